@@ -68,8 +68,8 @@ __global__ void __launch_bounds__(THREADS) paged_attention_mma_kernel(const Attn
   int lo = (p.window > 0) ? max(0, pos0 - p.window + 1) : 0;  // oldest key any row reads
   if (p.chunk > 0) lo = max(lo, (pos0 / p.chunk) * p.chunk);  // (the first token's chunk begins before the others')
   int hi = pos_last;                                          // newest key any row reads
-  if (SPLIT) {  // (single tokens: with chunks the splits count from the start of the token's chunk)
-    const int base = p.chunk > 0 ? (pos0 / p.chunk) * p.chunk : 0;
+  if (SPLIT) {  // (single tokens: with chunks the splits count from the start of the token's chunk, with a window from its first key's tile)
+    const int base = p.chunk > 0 ? (pos0 / p.chunk) * p.chunk : lo & ~(N_TILE - 1);
     lo = max(lo, base + split * p.split_keys);
     hi = min(hi, base + (split + 1) * p.split_keys - 1);
   }

@@ -54,6 +54,56 @@ extern "C" int llm_embed(const void* table, int table_dtype, const int* ids, flo
   return LLM_OK;
 }
 
+// The row of each token's id times `scale` plus a row of a second table that the token and the one before it in its request
+// choose: (previous * mul_prev + id * mul_cur) mod buckets, or row `buckets` for position 0. The token before a portion's first
+// one comes from `previous` [slots]; the block of that first token, the only one that reads the slot, also writes the portion's
+// last token there, after it has read it.
+template <typename T>
+__global__ void embed_pairs_kernel(const T* __restrict__ table, const T* __restrict__ pairs, int buckets, long long mul_prev, long long mul_cur,
+                                   float scale, const int* __restrict__ ids, const int* __restrict__ positions, const int* __restrict__ token_seq,
+                                   const int* __restrict__ seq_qoff, const int* __restrict__ seq_ntok, const int* __restrict__ seq_slot,
+                                   int* __restrict__ previous, float* __restrict__ out, int dim, int vocab) {
+  dep_launch();
+  dep_wait();
+  const int tok = blockIdx.x, seq = token_seq[tok], first = seq_qoff[seq];
+  int id = ids[tok];
+  if (id < 0 || id >= vocab) id = 0;  // ids are validated on the host; never read out of range
+  int row = buckets;
+  if (positions[tok] > 0) {
+    const int before = tok > first ? ids[tok - 1] : previous[seq_slot[seq]];
+    const long long mixed = ((long long)before * mul_prev + (long long)id * mul_cur) % buckets;
+    row = (int)(mixed < 0 ? mixed + buckets : mixed);
+  }
+  if (tok == first) {
+    __syncthreads();  // everyone has read the slot
+    if (threadIdx.x == 0) previous[seq_slot[seq]] = ids[first + max(seq_ntok[seq], 1) - 1];
+  }
+  const T* a = table + (size_t)id * dim;
+  const T* b = pairs + (size_t)row * dim;
+  float* dst = out + (size_t)tok * dim;
+  for (int i = threadIdx.x; i < dim; i += blockDim.x) dst[i] = fmaf(to_f32(a[i]), scale, to_f32(b[i]));
+}
+
+extern "C" int llm_embed_pairs(const void* table, const void* pairs, int dtype, int buckets, long long mul_prev, long long mul_cur, float scale,
+                               const int* ids, const int* positions, const int* token_seq, const int* seq_qoff, const int* seq_ntok,
+                               const int* seq_slot, int* previous, float* out, int n_tokens, int dim, int vocab, cudaStream_t stream) {
+  if (n_tokens == 0) return LLM_OK;
+  LLM_REQUIRE(n_tokens > 0 && dim > 0 && vocab > 0 && buckets > 0, "embed_pairs: bad sizes tokens=%d dim=%d vocab=%d buckets=%d", n_tokens, dim, vocab, buckets);
+  // products of an id and a multiplier, and their sum, stay far inside 64 bits
+  LLM_REQUIRE(mul_prev >= 0 && mul_cur >= 0 && mul_prev < (1ll << 31) && mul_cur < (1ll << 31), "embed_pairs: multipliers are not in 0 .. 2^31 - 1");
+  const int threads = dim >= 1024 ? 256 : 128;
+  if (dtype == LLM_F32)
+    launch_kernel(embed_pairs_kernel<float>, n_tokens, threads, 0, stream, (const float*)table, (const float*)pairs, buckets, mul_prev, mul_cur, scale,
+                  ids, positions, token_seq, seq_qoff, seq_ntok, seq_slot, previous, out, dim, vocab);
+  else if (dtype == LLM_BF16)
+    launch_kernel(embed_pairs_kernel<bf16>, n_tokens, threads, 0, stream, (const bf16*)table, (const bf16*)pairs, buckets, mul_prev, mul_cur, scale,
+                  ids, positions, token_seq, seq_qoff, seq_ntok, seq_slot, previous, out, dim, vocab);
+  else
+    LLM_REQUIRE(false, "embed_pairs: unknown table dtype %d", dtype);
+  LLM_CHECK_LAUNCH("embed_pairs");
+  return LLM_OK;
+}
+
 // ------------------------------------------------------------------------------------ RMSNorm
 // One block per output row. Source row r = rows ? rows[blockIdx.x] : blockIdx.x.
 // x = h[r] + sum_p delta[p][r] (partials added in index order); if write_back, h[r] = x.

@@ -6,7 +6,9 @@
 //              once and one over all key heads', with a weight a number), rotation of the first rot_dims numbers of a head in the
 //              half-split layout from (cos, sin) tables, value mixing v <- (1 - lambda) v + lambda v_first with the values that
 //              an earlier layer of the same step left for these tokens (or leaving them), and the write of k and v into the
-//              token's page. Keys have dk numbers a head, values dv.
+//              token's page. Keys have dk numbers a head, values dv. Options (QkvOptions, qkv_prep_after_kernel): a bias on the q and
+//              k columns; pairs of neighbours (2i, 2i + 1) turning together; every head divided by its root mean square behind the
+//              rotation; values that are the keys before any norm and rotation (the product then has no value columns).
 //   attention  one warp a (token, query head): keys lo..pos of the request through its block table, lo = the later of the
 //              window's and the chunk's start (a chunk is [c * size, (c + 1) * size) in absolute positions); softmax in float32
 //              whose denominator also holds exp(sink[head]) (optional: a learned term of the denominator alone); the result times
@@ -182,8 +184,86 @@ __global__ void __launch_bounds__(512)
   }
 }
 
+// What a mixer may ask for beside the above: bias [H * dk + G * dk] (or null) added to the q and k columns; neighbours: the pairs of
+// the rotation are (2i, 2i + 1) instead of (i, i + rot_dims / 2); unit_rms: each head over its root mean square (eps inside the
+// root) after the rotation; keys_as_values: the values are the k columns with their bias (dv == dk, no v columns).
+struct QkvOptions {
+  const float* bias;
+  int neighbours, unit_rms, keys_as_values;
+};
+
+// A warp a head, as in qkv_prep_kernel; a head's numbers lie in shared memory from the sums to the store, a pair of the rotation is
+// one lane's.
+template <typename T>
+__global__ void __launch_bounds__(PREP_WARPS * 32)
+    qkv_prep_after_kernel(const float* __restrict__ parts, int n_parts, size_t pstride, int width, int H, int G, int dk, int dv, int rot_dims,
+                          const float* __restrict__ wq, const float* __restrict__ wk, float eps, const float* __restrict__ cos_t,
+                          const float* __restrict__ sin_t, const int* __restrict__ positions, const int* __restrict__ token_seq,
+                          const int* __restrict__ block_table, int max_blocks, T* __restrict__ q_out, long long ld_q, T* __restrict__ kcache,
+                          T* __restrict__ vcache, int page_size, const QkvOptions o) {
+  extern __shared__ float sh[];  // PREP_WARPS rows of dk
+  dep_launch();
+  dep_wait();
+  const int tok = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int pos = positions[tok];
+  const size_t row = (size_t)tok * width;
+  const int half = rot_dims / 2;
+  const float* cs = cos_t ? cos_t + (size_t)pos * half : nullptr;
+  const float* sn = sin_t ? sin_t + (size_t)pos * half : nullptr;
+  const int page = block_table[(size_t)token_seq[tok] * max_blocks + pos / page_size];
+  const int in_page = pos % page_size;
+  float* buf = sh + (size_t)warp * dk;
+  for (int head = blockIdx.y * PREP_WARPS + warp; head < H + G; head += gridDim.y * PREP_WARPS) {
+    const bool is_q = head < H;
+    const size_t col0 = (size_t)head * dk;  // key heads lie right behind the query heads, in the product as in the bias
+    const size_t slot = is_q ? 0 : ((size_t)page * G + (head - H)) * page_size + in_page;
+    const float* w = is_q ? wq : wk;
+    T* v_dst = (!is_q && o.keys_as_values && vcache) ? vcache + slot * dv : nullptr;
+    float ss = 0.f;
+    for (int d = lane; d < dk; d += 32) {
+      float v = parts_sum(parts, n_parts, pstride, row + col0 + d);
+      if (o.bias) v += o.bias[col0 + d];
+      if (v_dst) v_dst[d] = from_f32<T>(v);
+      buf[d] = v;
+      ss += v * v;
+    }
+    if (w) {
+      const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)dk + eps);
+      for (int d = lane; d < dk; d += 32) buf[d] = buf[d] * inv * w[d];  // the lane's own numbers
+    }
+    __syncwarp();
+    for (int i = lane; i < half; i += 32) {
+      const int a = o.neighbours ? 2 * i : i, b = o.neighbours ? 2 * i + 1 : i + half;
+      const float x = buf[a], y = buf[b], c = cs[i], s = sn[i];
+      buf[a] = x * c - y * s;
+      buf[b] = y * c + x * s;
+    }
+    __syncwarp();
+    float inv = 1.0f;
+    if (o.unit_rms) {
+      float rs = 0.f;
+      for (int d = lane; d < dk; d += 32) rs += buf[d] * buf[d];
+      inv = 1.0f / sqrtf(warp_sum(rs) / (float)dk + eps);
+    }
+    T* dst;
+    if (is_q) dst = q_out + (size_t)tok * ld_q + col0;
+    else dst = kcache ? kcache + slot * dk : nullptr;
+    if (dst)
+      for (int d = lane; d < dk; d += 32) dst[d] = from_f32<T>(o.unit_rms ? buf[d] * inv : buf[d]);
+    __syncwarp();
+  }
+  if (vcache && !o.keys_as_values) {
+    const size_t vcol0 = (size_t)(H + G) * dk;
+    for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < G * dv; i += gridDim.y * blockDim.x) {
+      const float v = parts_sum(parts, n_parts, pstride, row + vcol0 + i);
+      const int g = i / dv, d = i - g * dv;
+      vcache[(((size_t)page * G + g) * page_size + in_page) * dv + d] = from_f32<T>(v);
+    }
+  }
+}
+
 constexpr int WARPS = 4;
-constexpr int MAX_HD = 256;
+constexpr int MAX_HD = 512;
 
 template <typename T, int R>  // R = ceil(dv / 32) output registers a lane
 __global__ void __launch_bounds__(WARPS * 32)
@@ -278,7 +358,7 @@ extern "C" int llm_qkv_prep(const float* parts, int n_parts, long long pstride, 
                             const float* wq, const float* wk, float eps, const float* cos_t, const float* sin_t, const int* positions,
                             const int* token_seq, const int* block_table, int max_blocks, void* q_out, long long ld_q, void* kcache,
                             void* vcache, int page_size, int mix_role, const float* lambda, float* v_first, int dtype, int n_tokens,
-                            int norm_wide, cudaStream_t stream) {
+                            int norm_wide, const float* bias, int neighbours, int unit_rms, int keys_as_values, cudaStream_t stream) {
   // G 0: the product holds queries alone (a layer that reads another layer's keys and values): nothing is written to a cache.
   // norm_wide: wq [H * dk] and wk [G * dk], one RMS norm over each whole projection instead of one a head
   if (n_tokens == 0) return LLM_OK;
@@ -286,7 +366,10 @@ extern "C" int llm_qkv_prep(const float* parts, int n_parts, long long pstride, 
   LLM_REQUIRE(G > 0 || (kcache == nullptr && mix_role == 0), "qkv_prep: a product without keys and values writes none");
   LLM_REQUIRE(rot_dims >= 0 && rot_dims % 2 == 0 && rot_dims <= dk, "qkv_prep: %d rotated dimensions do not fit a head of %d", rot_dims, dk);
   LLM_REQUIRE(rot_dims == 0 || (cos_t && sin_t), "qkv_prep: rotation tables missing");
-  LLM_REQUIRE((size_t)(H + G) * dk + (size_t)G * dv <= (size_t)width, "qkv_prep: columns outside the product");
+  LLM_REQUIRE((size_t)(H + G) * dk + (keys_as_values ? 0 : (size_t)G * dv) <= (size_t)width, "qkv_prep: columns outside the product");
+  LLM_REQUIRE(!keys_as_values || (dk == dv && G > 0), "qkv_prep: values that are keys have the keys' size");
+  const bool after = bias || neighbours || unit_rms || keys_as_values;
+  LLM_REQUIRE(!after || (!norm_wide && mix_role == 0), "qkv_prep: biases, neighbouring pairs, norms behind the rotation and keys as values go with norms a head and no value mixing");
   LLM_REQUIRE((kcache == nullptr) == (vcache == nullptr), "qkv_prep: keys and values are written together");
   LLM_REQUIRE(mix_role == 0 || (v_first && (mix_role == 1 || (mix_role == 2 && lambda))), "qkv_prep: value mixing needs its buffer and weight");
   const size_t smem = (size_t)PREP_WARPS * dk * sizeof(float);
@@ -308,6 +391,19 @@ extern "C" int llm_qkv_prep(const float* parts, int n_parts, long long pstride, 
   }
   // few tokens: the heads of a token are spread over several blocks, so that the sums of many parts are read side by side
   dim3 grid(n_tokens, n_tokens >= 512 ? 1 : min(ceil_div(H + G, PREP_WARPS), 8));
+  if (after) {
+    const QkvOptions o{bias, neighbours, unit_rms, keys_as_values};
+#define LLM_PREP_AFTER(T)                                                                                                               \
+  launch_kernel(qkv_prep_after_kernel<T>, grid, PREP_WARPS * 32, smem, stream, parts, n_parts, (size_t)pstride, width, H, G, dk, dv,     \
+                rot_dims, wq, wk, eps, cos_t, sin_t, positions, token_seq, block_table, max_blocks, (T*)q_out, ld_q, (T*)kcache,          \
+                (T*)vcache, page_size, o)
+    if (dtype == LLM_F32) LLM_PREP_AFTER(float);
+    else if (dtype == LLM_BF16) LLM_PREP_AFTER(bf16);
+    else LLM_REQUIRE(false, "qkv_prep: unknown dtype %d", dtype);
+#undef LLM_PREP_AFTER
+    LLM_CHECK_LAUNCH("qkv_prep");
+    return LLM_OK;
+  }
 #define LLM_PREP(T)                                                                                                                  \
   launch_kernel(qkv_prep_kernel<T>, grid, PREP_WARPS * 32, smem, stream, parts, n_parts, (size_t)pstride, width, H, G, dk, dv,    \
                 rot_dims, wq, wk, eps, cos_t, sin_t, positions, token_seq, block_table, max_blocks, (T*)q_out, ld_q, (T*)kcache,       \
@@ -341,7 +437,8 @@ extern "C" int llm_gated_attention_simt(const void* q, long long ld_q, const voi
   if (dv <= 32) LLM_GA(T, 1);  \
   else if (dv <= 64) LLM_GA(T, 2); \
   else if (dv <= 128) LLM_GA(T, 4); \
-  else LLM_GA(T, 8)
+  else if (dv <= 256) LLM_GA(T, 8); \
+  else LLM_GA(T, 16)
   if (dtype == LLM_F32) { LLM_GA_R(float); }
   else if (dtype == LLM_BF16) { LLM_GA_R(bf16); }
   else LLM_REQUIRE(false, "attention: unknown dtype %d", dtype);

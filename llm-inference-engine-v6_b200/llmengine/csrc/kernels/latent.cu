@@ -61,8 +61,8 @@ __global__ void latent_prep_kernel(const float* __restrict__ parts, int n_parts,
     if (i < R) ssk += x * x;
   }
   ssq = block_sum(ssq, red);
-  ssk = block_sum(ssk, red);
-  const float iq = 1.0f / sqrtf(ssq / (float)Rq + eps), ik = 1.0f / sqrtf(ssk / (float)R + eps);
+  ssk = R > 0 ? block_sum(ssk, red) : 0.f;  // R 0: the product holds no latent (a layer that reads another layer's)
+  const float iq = 1.0f / sqrtf(ssq / (float)Rq + eps), ik = R > 0 ? 1.0f / sqrtf(ssk / (float)R + eps) : 0.f;
   T* q_out = cq + (size_t)tok * ld_cq;
   for (int i = threadIdx.x; i < Rq; i += blockDim.x) q_out[i] = from_f32<T>(row[i] * iq * wq[i]);
   if (cache == nullptr) return;
@@ -146,12 +146,13 @@ __device__ __forceinline__ bool rows_vectorizable(const T* a, long long lda, lon
          lda_h % per == 0 && ldw % per == 0;
 }
 
-// out[t, h*ldo_h + n] = (sum_k a[t, h*lda_h + k] * w[(h*N + n), k]) (* sigmoid(sum_p gate[p][t][g_off + h*N + n]))
+// out[t, h*ldo_h + n] = (sum_k a[t, h*lda_h + k] * w[(h*N + n), k]) (* sigmoid(sum_p gate[p][t][g_off + h*N + n]), or with g_head
+// one gate a head, column g_off + h)
 template <typename T>
 __global__ void __launch_bounds__(HP_WARPS * 32)
     heads_product_kernel(const T* __restrict__ a, long long lda, long long lda_h, const T* __restrict__ w, long long ldw,
                          T* __restrict__ out, long long ldo, long long ldo_h, int T_, int N, int K,
-                         const float* __restrict__ gate, int n_parts, size_t pstride, int gwidth, int g_off) {
+                         const float* __restrict__ gate, int n_parts, size_t pstride, int gwidth, int g_off, int g_head) {
   dep_launch();
   dep_wait();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -165,7 +166,7 @@ __global__ void __launch_bounds__(HP_WARPS * 32)
     for (int i = 0; i < HP_TOKENS; ++i)
       if (i == lane) v = acc[i];
     if (gate) {
-      const float g = sum_parts(gate, n_parts, pstride, (size_t)(t0 + lane) * gwidth + g_off + (size_t)h * N + n);
+      const float g = sum_parts(gate, n_parts, pstride, (size_t)(t0 + lane) * gwidth + g_off + (g_head ? (size_t)h : (size_t)h * N + n));
       v *= 1.0f / (1.0f + expf(-g));
     }
     out[(size_t)(t0 + lane) * ldo + (size_t)h * ldo_h + n] = from_f32<T>(v);
@@ -247,7 +248,8 @@ template <typename T, int NV>
 __global__ void __launch_bounds__(LA_WARPS * 32)
     latent_attention_simt_kernel(const T* __restrict__ ql, const T* __restrict__ cache, const int* __restrict__ positions,
                                  const int* __restrict__ token_seq, const int* __restrict__ block_table, int max_blocks,
-                                 T* __restrict__ out, int n_tokens, int H, int R, int dr, int page_size, float scale, int window) {
+                                 T* __restrict__ out, int n_tokens, int H, int R, int dr, int page_size, float scale, int window,
+                                 const float* __restrict__ sink) {
   extern __shared__ float q_s[];  // LA_WARPS x (R + dr)
   dep_launch();
   dep_wait();
@@ -299,6 +301,14 @@ __global__ void __launch_bounds__(LA_WARPS * 32)
     }
     m = m_new;
   }
+  if (sink) {  // one more term of the denominator, with no value; not scaled
+    const float sk = sink[head];
+    const float m_new = fmaxf(m, sk);
+    const float alpha = expf(m - m_new);
+    l = l * alpha + expf(sk - m_new);
+#pragma unroll
+    for (int i = 0; i < NV; ++i) acc[i] *= alpha;
+  }
   const float inv = 1.0f / l;
   T* o = out + ((size_t)tok * H + head) * R;
 #pragma unroll
@@ -330,7 +340,7 @@ extern "C" int llm_latent_prep(const float* parts, int n_parts, long long pstrid
                                int max_blocks, void* cq, long long ld_cq, void* cache, int page_size, int dtype, int n_tokens,
                                cudaStream_t stream) {
   if (n_tokens == 0) return LLM_OK;
-  LLM_REQUIRE(n_tokens > 0 && n_parts >= 1 && Rq > 0 && R > 0 && dr >= 0, "latent_prep: bad sizes");
+  LLM_REQUIRE(n_tokens > 0 && n_parts >= 1 && Rq > 0 && R >= 0 && dr >= 0 && (R > 0 || (cache == nullptr && dr == 0)), "latent_prep: bad sizes");
   LLM_REQUIRE(rot_dims >= 0 && rot_dims % 2 == 0 && rot_dims <= dr, "latent_prep: %d rotated dimensions do not fit a part of %d", rot_dims, dr);
   LLM_REQUIRE(q_off >= 0 && kv_off >= 0 && q_off + Rq <= width && kv_off + R + dr <= width, "latent_prep: columns outside the product");
   LLM_REQUIRE(rot_dims == 0 || (cos_t && sin_t), "latent_prep: rotation tables missing");
@@ -350,17 +360,17 @@ extern "C" int llm_latent_prep(const float* parts, int n_parts, long long pstrid
 
 extern "C" int llm_heads_product(const void* a, long long lda, long long lda_h, const void* w, long long ldw, void* out, long long ldo,
                                  long long ldo_h, int n_tokens, int H, int N, int K, const float* gate, int n_parts, long long pstride,
-                                 int gwidth, int g_off, int dtype, cudaStream_t stream) {
+                                 int gwidth, int g_off, int g_head, int dtype, cudaStream_t stream) {
   if (n_tokens == 0) return LLM_OK;
   LLM_REQUIRE(n_tokens > 0 && H > 0 && N > 0 && K > 0 && H <= 65535, "heads_product: bad sizes");
   LLM_REQUIRE(ceil_div(n_tokens, HP_TOKENS) <= 65535, "heads_product: %d tokens are too many for one launch", n_tokens);
   dim3 grid(ceil_div(N, HP_WARPS), H, ceil_div(n_tokens, HP_TOKENS));
   if (dtype == LLM_F32)
     launch_kernel(heads_product_kernel<float>, grid, HP_WARPS * 32, 0, stream, (const float*)a, lda, lda_h, (const float*)w, ldw, (float*)out,
-                  ldo, ldo_h, n_tokens, N, K, gate, n_parts, (size_t)pstride, gwidth, g_off);
+                  ldo, ldo_h, n_tokens, N, K, gate, n_parts, (size_t)pstride, gwidth, g_off, g_head);
   else if (dtype == LLM_BF16)
     launch_kernel(heads_product_kernel<bf16>, grid, HP_WARPS * 32, 0, stream, (const bf16*)a, lda, lda_h, (const bf16*)w, ldw, (bf16*)out,
-                  ldo, ldo_h, n_tokens, N, K, gate, n_parts, (size_t)pstride, gwidth, g_off);
+                  ldo, ldo_h, n_tokens, N, K, gate, n_parts, (size_t)pstride, gwidth, g_off, g_head);
   else
     LLM_REQUIRE(false, "heads_product: unknown dtype %d", dtype);
   LLM_CHECK_LAUNCH("heads_product");
@@ -405,7 +415,7 @@ extern "C" int llm_latent_query(const void* q, long long ldq, const void* wkt, v
 
 extern "C" int llm_latent_attention_simt(const void* ql, const void* cache, int dtype, const int* positions, const int* token_seq,
                                          const int* block_table, int max_blocks, void* out, int n_tokens, int H, int R, int dr,
-                                         int page_size, float scale, int window, cudaStream_t stream) {
+                                         int page_size, float scale, int window, const float* sink, cudaStream_t stream) {
   if (n_tokens == 0) return LLM_OK;
   LLM_REQUIRE(n_tokens > 0 && H > 0 && R > 0 && dr >= 0, "latent_attention: bad sizes");
   LLM_REQUIRE(R <= 1024, "latent_attention: a latent of %d numbers is more than the CUDA-core kernel keeps (1024)", R);
@@ -415,7 +425,7 @@ extern "C" int llm_latent_attention_simt(const void* ql, const void* cache, int 
   const int grid = ceil_div((long long)n_tokens * H, LA_WARPS);
 #define LLM_LA_CASE(T, NV)                                                                                                        \
   launch_kernel(latent_attention_simt_kernel<T, NV>, grid, LA_WARPS * 32, smem, stream, (const T*)ql, (const T*)cache, positions, \
-                token_seq, block_table, max_blocks, (T*)out, n_tokens, H, R, dr, page_size, scale, window)
+                token_seq, block_table, max_blocks, (T*)out, n_tokens, H, R, dr, page_size, scale, window, sink)
 #define LLM_LA_SIZES(T)              \
   if (R <= 64) LLM_LA_CASE(T, 2);    \
   else if (R <= 128) LLM_LA_CASE(T, 4); \

@@ -13,7 +13,9 @@
 // the value columns, R/4 accumulator columns a warp. Each row is masked by its own token's position (and
 // window): the result for a token does not depend on what else is in the step.
 // For decoding the key range is also cut into splits of a fixed number of keys (absolute boundaries); every
-// split writes a normalised partial output with its (max, sum), and a second kernel merges them in index order.
+// split writes a normalised partial output with its (max, sum), and a second kernel merges them in index order. With a window
+// the splits are counted from the window's first key, rounded down to a multiple of 64. A sink (a float per head whose
+// exponential is one more term of the denominator) is added behind the keys, or where the splits are merged.
 #include "common.cuh"
 #include "mma_common.cuh"
 
@@ -30,6 +32,7 @@ struct LatentParams {
   const bf16* cache;  // [pages, page_size, Dk]
   const int* seq_start; const int* seq_ntok; const int* seq_qoff; const int* block_table;
   int max_blocks, H, gh, n_htiles, R, Dk, page_size, window;
+  const float* sink;  // [H] or null
   float scale;
   bf16* out;          // [tokens, H, R]
   float* part_o; float* part_ml; int split_keys, n_splits; long long n_tokens;
@@ -70,8 +73,9 @@ __global__ void __launch_bounds__(RGS * 128) latent_attention_mma_kernel(const L
   int lo = (p.window > 0) ? max(0, pos0 - p.window + 1) : 0;
   int hi = pos_last;
   if (SPLIT) {
-    lo = max(lo, split * p.split_keys);
-    hi = min(hi, (split + 1) * p.split_keys - 1);
+    const int base = lo & ~63;  // (single tokens: 0, or near the window's first key)
+    lo = max(lo, base + split * p.split_keys);
+    hi = min(hi, base + (split + 1) * p.split_keys - 1);
   }
   const int* table = p.block_table + (size_t)seq * p.max_blocks;
   auto row_valid = [&](int r) { return r < n_tq * gh && head0 + r % gh < p.H; };
@@ -262,6 +266,19 @@ __global__ void __launch_bounds__(RGS * 128) latent_attention_mma_kernel(const L
   }
   cp_async_wait<0>();
 
+  if (!SPLIT && p.sink != nullptr) {  // one more term of the denominator (scores are in units of log2(e); the sink is not scaled)
+    const float sk_a = p.sink[min(head0 + row_a % gh, p.H - 1)] * 1.4426950408889634f;
+    const float sk_b = p.sink[min(head0 + row_b % gh, p.H - 1)] * 1.4426950408889634f;
+    const float mn_a = fmaxf(m_a, sk_a), mn_b = fmaxf(m_b, sk_b);
+    const float al_a = exp2f(m_a - mn_a), al_b = exp2f(m_b - mn_b);
+    l_a = l_a * al_a + exp2f(sk_a - mn_a);
+    l_b = l_b * al_b + exp2f(sk_b - mn_b);
+#pragma unroll
+    for (int d = 0; d < 2 * DT; ++d) {
+      o_acc[d][0] *= al_a; o_acc[d][1] *= al_a;
+      o_acc[d][2] *= al_b; o_acc[d][3] *= al_b;
+    }
+  }
   // ---- write: rows a and b of this thread, columns 2*(lane%4)+{0,1} of every 8-wide tile of this warp's quarter
   const float inv_a = l_a > 0.f ? 1.f / l_a : 0.f, inv_b = l_b > 0.f ? 1.f / l_b : 0.f;
 #pragma unroll
@@ -295,7 +312,7 @@ __global__ void __launch_bounds__(RGS * 128) latent_attention_mma_kernel(const L
 constexpr int LC_THREADS = 256, LC_MAX_SPLITS = 128;
 __global__ void __launch_bounds__(LC_THREADS)
     latent_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml, int n_splits, long long n_tokens, int H,
-                          int R, bf16* __restrict__ out) {
+                          int R, bf16* __restrict__ out, const float* __restrict__ sink) {
   __shared__ float w_s[LC_MAX_SPLITS];
   __shared__ float red[33];
   dep_launch();
@@ -315,10 +332,13 @@ __global__ void __launch_bounds__(LC_THREADS)
   mx = red[0];
 #pragma unroll
   for (int i = 1; i < LC_THREADS / 32; ++i) mx = fmaxf(mx, red[i]);
+  const float sk = sink ? sink[item % H] * 1.4426950408889634f : -INFINITY;  // (the splits' maxima are in units of log2(e))
+  mx = fmaxf(mx, sk);
   if (tid < LC_MAX_SPLITS) w_s[tid] = (tid < n_splits && m != -INFINITY) ? l * exp2f(m - mx) : 0.f;
   __syncthreads();
   float den = 0.f;
   for (int s = 0; s < n_splits; ++s) den += w_s[s];  // index order, the same in every thread
+  if (sink) den += exp2f(sk - mx);
   const float inv = den > 0.f ? 1.f / den : 0.f;
   for (int d = tid; d < R; d += LC_THREADS) {
     float acc = 0.f;
@@ -373,7 +393,7 @@ extern "C" long long llm_latent_attention_scratch_floats(int n_tokens, int H, in
 extern "C" int llm_latent_attention_mma(const void* ql, const void* cache, const int* seq_start, const int* seq_ntok,
                                         const int* seq_qoff, const int* block_table, int max_blocks, void* out, int n_seqs,
                                         int n_tokens, int max_new_tokens, int H, int R, int dr, int page_size, float scale, int window,
-                                        int n_splits, int split_keys, float* scratch, cudaStream_t stream) {
+                                        int n_splits, int split_keys, float* scratch, const float* sink, cudaStream_t stream) {
   if (n_tokens == 0 || n_seqs == 0) return LLM_OK;
   LLM_REQUIRE(llm_latent_attention_mma_supported(H, R, dr), "latent_attention_mma: geometry not supported (heads=%d latent=%d rotated=%d)", H, R, dr);
   LLM_REQUIRE(page_size > 0 && max_blocks > 0 && window >= 0 && max_new_tokens > 0, "latent_attention_mma: bad sizes");
@@ -390,7 +410,7 @@ extern "C" int llm_latent_attention_mma(const void* ql, const void* cache, const
   const int rows = lm_rows(wide ? 4 : (split && H <= 16 ? 1 : 2));
   p.block_table = block_table; p.max_blocks = max_blocks; p.H = H; p.gh = H < rows ? H : rows;
   p.n_htiles = (H + p.gh - 1) / p.gh; p.R = R; p.Dk = R + dr; p.page_size = page_size; p.window = window; p.scale = scale;
-  p.out = (bf16*)out; p.n_splits = n_splits; p.split_keys = split_keys; p.n_tokens = n_tokens;
+  p.out = (bf16*)out; p.n_splits = n_splits; p.split_keys = split_keys; p.n_tokens = n_tokens; p.sink = sink;
   p.part_o = scratch; p.part_ml = scratch ? scratch + (size_t)n_splits * n_tokens * H * R : nullptr;
   const int tq_cap = rows / p.gh;
   LLM_REQUIRE((long long)n_seqs <= 65535 && (long long)p.n_htiles * n_splits <= 65535, "latent_attention_mma: batch too large for the grid");
@@ -410,7 +430,7 @@ extern "C" int llm_latent_attention_mma(const void* ql, const void* cache, const
   if (split) {
     const long long items = (long long)n_tokens * H;
     launch_kernel(latent_combine_kernel, (int)items, LC_THREADS, 0, stream, (const float*)p.part_o, (const float*)p.part_ml, n_splits,
-                  (long long)n_tokens, H, R, (bf16*)out);
+                  (long long)n_tokens, H, R, (bf16*)out, sink);
   }
   LLM_CHECK_LAUNCH("latent_attention_mma");
   return LLM_OK;

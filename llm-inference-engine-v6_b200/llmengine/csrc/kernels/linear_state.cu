@@ -1,10 +1,11 @@
 // Mixers whose memory is a matrix per head ("linear state"): S [dk, dv] per request and head, float32, kept in the request's state
-// slot, updated token after token by a rank-one write k v^T and read by a query. Three update rules share one kernel:
+// slot, updated token after token by a rank-one write k v^T and read by a query. Four update rules share one kernel:
 //
 //   MODE 0  decay a key channel, write, read:   S <- diag(a_t) S + k_t v_t^T;              o_t = S^T q_t
 //   MODE 1  read with a bonus, decay, write:    o_t = (S + diag(u) k_t v_t^T)^T q_t;       S <- diag(a_t) S + k_t v_t^T
 //   MODE 2  delta rule with a decay a head:     S <- g_t S;  w = beta_t (v_t - S^T k_t);   S <- S + k_t w^T;   o_t = S^T q_t
 //           (q and k made unit vectors per head first: x / sqrt(sum x^2 + unit_eps))
+//   MODE 3  delta rule with a decay a channel:  S <- diag(a_t) S;  the rest as MODE 2, beta_t = sigmoid of its product's sums
 //
 // Every column S[:, j] evolves by itself, so a block takes a (request, head, tile of columns) and walks the request's tokens of the
 // step in order; a column's dk numbers are spread over R lanes of a warp (KPT = 16 numbers a lane), the two dot products of a
@@ -17,9 +18,11 @@
 // S[channel_of(m, r, R), j]; loads and stores of a warp are then 128 contiguous bytes. R = the power of two >= dk / 16.
 //
 // Beside it: token_shift (every projection's own blend of a token's input with the previous token's, the previous token of a
-// portion's first token coming from the slot), delta_gates (the delta rule's decay and write strength per head) and
-// head_norm_gate (every head's result divided by its root mean square, times a weight, times silu of a gate).
+// portion's first token coming from the slot), delta_gates (the delta rule's decay and write strength per head), channel_gates
+// (two low-rank maps at once: a decay per head and key channel, and the gate of the result) and head_norm_gate (every head's
+// result divided by its root mean square, times a weight, times silu or sigmoid of a gate).
 #include "common.cuh"
+#include "mma_common.cuh"
 
 #include <cmath>
 
@@ -42,8 +45,8 @@ struct Sums {  // columns off.. of float32 sums [parts, rows, width]
 };
 
 struct LinearStateParams {
-  Sums q, k, v;
-  const float* decay; int decay_width, decay_off;  // float32 rows: MODE 0/1 a number a (head, key channel); MODE 2 [g: H | beta: H]
+  Sums q, k, v, b;                                 // b: MODE 3, one number a head (before its sigmoid)
+  const float* decay; int decay_width, decay_off;  // float32 rows: MODE 0/1/3 a number a (head, key channel); MODE 2 [g: H | beta: H]
   const float* bonus;                              // MODE 1: [H, dk]
   float* state;                                    // [slots, H, R * KPT, dv] in the layout above
   const int* seq_qoff; const int* seq_ntok; const int* seq_slot;
@@ -78,8 +81,9 @@ __device__ __forceinline__ float lanes_sum(float x) {  // over the R lanes of a 
 struct TileRows {  // a tile of tokens in shared memory
   float* q;  // [tile][dkp]
   float* k;  // [tile][dkp]
-  float* a;  // [tile][dkp] (MODE 0/1) or [tile][2] (MODE 2)
+  float* a;  // [tile][dkp] (MODE 0/1/3) or [tile][2] (MODE 2)
   float* v;  // [tile][dv]
+  float* b;  // [tile] (MODE 3)
 };
 
 // A tile of tokens through the rule: s the thread's numbers of its column, v[tt * dv + col] the column's value; out points at the
@@ -101,6 +105,7 @@ __device__ __forceinline__ void walk_tile(float (&s)[KPT], const float (&u)[KPT]
       g_ = rows.a[tt * a_stride];
       b_ = rows.a[tt * a_stride + 1];
     }
+    if (MODE == 3) b_ = rows.b[tt];
     v_ = live ? rows.v[tt * dv + col] : 0.f;
   };
   read(0, kk, qq, aa, vj, g, beta);
@@ -127,7 +132,7 @@ __device__ __forceinline__ void walk_tile(float (&s)[KPT], const float (&u)[KPT]
       float dot[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
       for (int m = 0; m < KPT; ++m) {
-        s[m] *= g;
+        s[m] *= MODE == 3 ? aa[m] : g;
         dot[m & 3] = fmaf(s[m], kk[m], dot[m & 3]);
       }
       const float d = lanes_sum<R>((dot[0] + dot[1]) + (dot[2] + dot[3]));
@@ -176,7 +181,7 @@ __device__ __forceinline__ void copies_wait_but_last() { asm volatile("cp.async.
 template <int MODE>
 __device__ __forceinline__ void fetch_issue(const LinearStateParams& p, size_t row0, int cnt, int head, int kvh, int dk, int dkp, int dv,
                                             int tid, int n_thr, const TileRows& rows) {
-  const bool unit = MODE == 2 && p.unit_eps >= 0.f;
+  const bool unit = MODE >= 2 && p.unit_eps >= 0.f;
   const float qmul = unit ? 1.0f : p.q_scale;
   const int lg = __ffs(dkp) - 1;  // dkp is a power of two
   const int n_qk = cnt * dkp, n_v = cnt * dv;
@@ -222,6 +227,8 @@ __device__ __forceinline__ void fetch_issue(const LinearStateParams& p, size_t r
     if (MODE == 2)
       for (int e = tid; e < 2 * cnt; e += n_thr)
         copy4_async(rows.a + e, p.decay + (row0 + (e >> 1)) * p.decay_width + p.decay_off + (e & 1) * p.H + head);
+    if (MODE == 3)
+      for (int e = tid; e < cnt; e += n_thr) copy4_async(rows.b + e, p.b.p + (row0 + e) * p.b.width + p.b.off + head);
     return;
   }
   constexpr int U = 4;  // elements a thread has in flight: their loads are issued together, part after part in the parts' order
@@ -278,12 +285,16 @@ __device__ __forceinline__ void fetch_issue(const LinearStateParams& p, size_t r
   }
   if (MODE == 2)
     for (int e = tid; e < 2 * cnt; e += n_thr) rows.a[e] = p.decay[(row0 + (e >> 1)) * p.decay_width + p.decay_off + (e & 1) * p.H + head];
+  if (MODE == 3)
+    for (int e = tid; e < cnt; e += n_thr) rows.b[e] = parts_sum(p.b.p, p.b.n, p.b.stride, (row0 + e) * p.b.width + p.b.off + head);
 }
 
 template <int MODE>
 __device__ __forceinline__ void fetch_finish(const LinearStateParams& p, int cnt, int dk, int dkp, int tid, int n_thr, const TileRows& rows) {
-  const bool unit = MODE == 2 && p.unit_eps >= 0.f;
+  const bool unit = MODE >= 2 && p.unit_eps >= 0.f;
   const float qmul = unit ? 1.0f : p.q_scale;
+  if (MODE == 3)  // the thread's own numbers, as fetch_issue dealt them
+    for (int e = tid; e < cnt; e += n_thr) rows.b[e] = 1.0f / (1.0f + expf(-rows.b[e]));
   if (p.one_part && qmul != 1.0f) {  // the thread's own copies, as fetch_issue dealt them
     const int n_qk = cnt * dkp;
     if (p.vec4) {
@@ -338,13 +349,14 @@ __global__ void __launch_bounds__(LS_BLOCK, FEW ? 2 : 1) linear_state_kernel(con
   const bool live = walker && col < dv;
   const int tile = p.tile, n_tiles = (n_tok + tile - 1) / tile;
   const size_t a_floats = ((size_t)tile * a_stride + 3) & ~(size_t)3;
-  const size_t buf_floats = ((size_t)tile * (2 * dkp + dv) + a_floats + 3) & ~(size_t)3;  // every region starts on 16 bytes
+  const size_t buf_floats = ((size_t)tile * (2 * dkp + dv + (MODE == 3 ? 1 : 0)) + a_floats + 3) & ~(size_t)3;  // every region but the last starts on 16 bytes
   auto rows_of = [&](int i) {
     TileRows r;
     r.q = sh_ls + (size_t)(i % LS_BUFFERS) * buf_floats;
     r.k = r.q + (size_t)tile * dkp;
     r.a = r.k + (size_t)tile * dkp;
     r.v = r.a + a_floats;
+    r.b = r.v + (size_t)tile * dv;
     return r;
   };
   const int ftid = threadIdx.x - p.walkers, n_fetch = LS_FETCHERS;
@@ -436,11 +448,74 @@ __global__ void delta_gates_kernel(const Sums a, const Sums b, const float* __re
   out[tok * 2 * H + H + h] = 1.0f / (1.0f + expf(-parts_sum(b.p, b.n, b.stride, tok * b.width + b.off + h)));
 }
 
-// a warp a (token, head): out = o / sqrt(mean(o^2) + eps) * weight * silu(gate); weight [dv] for all heads or [H * dv]
+// Two low-rank maps of one product's sums in one launch. Columns x0.off .. + R0 of the sums feed map 0, the decay of a delta rule
+// with a decay per key channel: out0[t, c] = exp(-exp(a_log[c / per]) * softplus(bias0[c] + sum_r w0[c, r] x0[t, r])); columns
+// x1.off .. + R1 feed map 1, out1[t, c] = sum_r w1[c, r] x1[t, r], the sums of the result's gate. All float32.
+struct ChannelGates {
+  Sums x0, x1;
+  int R0, R1, C0, C1, per;
+  const float* bias0; const float* a_log;
+  float* out0; float* out1;
+  int n_tokens;
+};
+
+__device__ __forceinline__ float channel_decay(float z, float a_log) {
+  return expf(-expf(a_log) * (z > 20.0f ? z : log1pf(expf(z))));
+}
+
+// A block: 32 channels of one map x 8 tokens; its four warps take a quarter of the rank each, warp 0 adds the quarters in index
+// order. wt: the maps stored transposed [R, C] (neighbouring channels read neighbouring words).
+template <typename T>
+__global__ void __launch_bounds__(128) channel_gates_kernel(const ChannelGates p, const T* __restrict__ wt0, const T* __restrict__ wt1) {
+  extern __shared__ __align__(16) float sm_cg[];  // low [R][8], then quarters [4][32][8]
+  dep_launch();
+  dep_wait();
+  const int blocks0 = (p.C0 + 31) / 32;
+  const bool first = (int)blockIdx.x < blocks0;
+  const Sums x = first ? p.x0 : p.x1;
+  const T* wt = first ? wt0 : wt1;
+  const int R = first ? p.R0 : p.R1, C = first ? p.C0 : p.C1, c0 = ((int)blockIdx.x - (first ? 0 : blocks0)) * 32;
+  float* low = sm_cg;
+  float* quarter = sm_cg + (size_t)R * 8;
+  const int t0 = blockIdx.y * 8;
+  for (int i = threadIdx.x; i < 8 * R; i += 128) {
+    const int tl = i / R, r = i - tl * R;
+    low[r * 8 + tl] = t0 + tl < p.n_tokens ? parts_sum(x.p, x.n, x.stride, (size_t)(t0 + tl) * x.width + x.off + r) : 0.f;
+  }
+  __syncthreads();
+  const int lane = threadIdx.x & 31, part = threadIdx.x >> 5;
+  const int c = min(c0 + lane, C - 1);
+  const int per = (R + 3) / 4, r_end = min(R, (part + 1) * per);
+  float acc[8];
+#pragma unroll
+  for (int i = 0; i < 8; ++i) acc[i] = 0.f;
+#pragma unroll 8
+  for (int r = part * per; r < r_end; ++r) {
+    const float wv = to_f32(wt[(size_t)r * C + c]);
+    const float4 v0 = *reinterpret_cast<const float4*>(low + r * 8), v1 = *reinterpret_cast<const float4*>(low + r * 8 + 4);
+    acc[0] = fmaf(wv, v0.x, acc[0]); acc[1] = fmaf(wv, v0.y, acc[1]); acc[2] = fmaf(wv, v0.z, acc[2]); acc[3] = fmaf(wv, v0.w, acc[3]);
+    acc[4] = fmaf(wv, v1.x, acc[4]); acc[5] = fmaf(wv, v1.y, acc[5]); acc[6] = fmaf(wv, v1.z, acc[6]); acc[7] = fmaf(wv, v1.w, acc[7]);
+  }
+#pragma unroll
+  for (int i = 0; i < 8; ++i) quarter[(part * 32 + lane) * 8 + i] = acc[i];
+  __syncthreads();
+  if (c0 + lane >= C) return;
+  const float b = first ? p.bias0[c] : 0.f, al = first ? p.a_log[c / p.per] : 0.f;
+  for (int i = part; i < 8; i += 4) {  // every warp finishes two of the tokens
+    const int t = t0 + i;
+    if (t >= p.n_tokens) break;
+    const float z = ((quarter[lane * 8 + i] + quarter[(32 + lane) * 8 + i]) + quarter[(64 + lane) * 8 + i]) + quarter[(96 + lane) * 8 + i] + b;
+    if (first) p.out0[(size_t)t * C + c] = channel_decay(z, al);
+    else p.out1[(size_t)t * C + c] = z;
+  }
+}
+
+// a warp a (token, head): out = o / sqrt(mean(o^2) + eps) * weight * act(gate), act silu or sigmoid; weight [dv] for all heads or
+// [H * dv]
 template <typename T>
 __global__ void __launch_bounds__(128)
     head_norm_gate_kernel(const float* __restrict__ o, const float* __restrict__ weight, int weight_per_head, const Sums gate, float eps,
-                          T* __restrict__ out, int n_tokens, int H, int dv) {
+                          T* __restrict__ out, int n_tokens, int H, int dv, int sigmoid) {
   dep_launch();
   dep_wait();
   const long long item = (long long)blockIdx.x * 4 + (threadIdx.x >> 5);
@@ -457,7 +532,7 @@ __global__ void __launch_bounds__(128)
     float v = row[d] * inv * weight[weight_per_head ? (size_t)head * dv + d : d];
     if (gate.p) {
       const float g = parts_sum(gate.p, gate.n, gate.stride, tok * gate.width + gate.off + (size_t)head * dv + d);
-      v *= g / (1.0f + expf(-g));
+      v *= (sigmoid ? 1.0f : g) / (1.0f + expf(-g));
     }
     out[tok * (size_t)H * dv + (size_t)head * dv + d] = from_f32<T>(v);
   }
@@ -512,21 +587,23 @@ extern "C" int llm_linear_state_lanes(int dk) {
 }
 
 extern "C" int llm_linear_state(int mode, const float* q, int qn, long long qs, int qw, int qo, const float* k, int kn, long long ks, int kw,
-                                int ko, const float* v, int vn, long long vs, int vw, int vo, const float* decay, int decay_width,
-                                int decay_off, const float* bonus, float* state, const int* seq_qoff, const int* seq_ntok,
+                                int ko, const float* v, int vn, long long vs, int vw, int vo, const float* b, int bn, long long bs, int bw,
+                                int bo, const float* decay, int decay_width, int decay_off, const float* bonus, float* state, const int* seq_qoff, const int* seq_ntok,
                                 const int* seq_slot, float* out, int n_tokens, int n_seqs, int H, int G, int dk, int dv, float q_scale,
                                 float unit_eps, int decay_const, cudaStream_t stream) {
   // decay_const: `decay` is one row that holds for every token (decays that are constants of the model)
   if (n_seqs == 0) return LLM_OK;
-  LLM_REQUIRE(mode >= 0 && mode <= 2, "linear_state: unknown update rule %d", mode);
+  LLM_REQUIRE(mode >= 0 && mode <= 3, "linear_state: unknown update rule %d", mode);
   LLM_REQUIRE(n_seqs > 0 && n_seqs <= 65535 && H > 0 && H <= 65535 && G > 0 && H % G == 0 && dv > 0, "linear_state: bad sizes");
   LLM_REQUIRE(llm_linear_state_lanes(dk) > 0, "linear_state: a key size of %d is not in 1..%d", dk, 32 * KPT);
-  LLM_REQUIRE(mode == 2 || G == H, "linear_state: only the delta rule shares query/key heads");
+  LLM_REQUIRE(mode >= 2 || G == H, "linear_state: only the delta rules share query/key heads");
+  LLM_REQUIRE(mode != 3 || (b && bn >= 1 && bo >= 0 && bo + H <= bw), "linear_state: the delta rule with a decay a channel needs the sums of beta");
   LLM_REQUIRE(q && k && v && decay && state && out && qn >= 1 && kn >= 1 && vn >= 1 && (mode != 1 || bonus), "linear_state: missing tensors");
   LLM_REQUIRE(qo + G * dk <= qw && ko + G * dk <= kw && vo + H * dv <= vw && decay_off + (mode == 2 ? 2 * H : H * dk) <= decay_width,
               "linear_state: columns outside their rows");
   LinearStateParams p;
   p.q = Sums{q, qn, (size_t)qs, qw, qo}; p.k = Sums{k, kn, (size_t)ks, kw, ko}; p.v = Sums{v, vn, (size_t)vs, vw, vo};
+  p.b = Sums{b, bn, (size_t)bs, bw, bo};
   p.decay = decay; p.decay_width = decay_const ? 0 : decay_width; p.decay_off = decay_off; p.bonus = bonus; p.state = state;
   p.seq_qoff = seq_qoff; p.seq_ntok = seq_ntok; p.seq_slot = seq_slot; p.out = out;
   p.H = H; p.G = G; p.dk = dk; p.dv = dv; p.R = lanes_for(dk); p.q_scale = q_scale; p.unit_eps = unit_eps;
@@ -534,13 +611,13 @@ extern "C" int llm_linear_state(int mode, const float* q, int qn, long long qs, 
   const int a_stride = mode == 2 ? 2 : dkp;
   auto smem_for = [&](int tile) {  // as the kernel lays a buffer out
     const size_t a_floats = ((size_t)tile * a_stride + 3) & ~(size_t)3;
-    return LS_BUFFERS * ((((size_t)tile * (2 * dkp + dv) + a_floats + 3) & ~(size_t)3) * sizeof(float));
+    return LS_BUFFERS * ((((size_t)tile * (2 * dkp + dv + (mode == 3 ? 1 : 0)) + a_floats + 3) & ~(size_t)3) * sizeof(float));
   };
   const bool few = n_tokens <= 2 * n_seqs;
   p.tile = few ? 2 : 16;
   while (p.tile > 1 && smem_for(p.tile) > 48 * 1024) p.tile /= 2;
   LLM_REQUIRE(smem_for(p.tile) <= 48 * 1024, "linear_state: heads of %d / %d numbers exceed one block's shared memory", dk, dv);
-  p.one_part = qn == 1 && kn == 1 && vn == 1;
+  p.one_part = qn == 1 && kn == 1 && vn == 1 && (mode != 3 || bn == 1);
   auto quads = [](const void* ptr, long long width, long long off) { return ((uintptr_t)ptr & 15) == 0 && width % 4 == 0 && off % 4 == 0; };
   p.vec4 = dk % 4 == 0 && dv % 4 == 0 && quads(q, qw, qo) && quads(k, kw, ko) && quads(v, vw, vo) && (mode == 2 || quads(decay, p.decay_width, decay_off));
   // the walk is bound by what a multiprocessor's shared memory delivers a token, so few blocks are cut into more, down to a warp of walkers
@@ -561,7 +638,7 @@ extern "C" int llm_linear_state(int mode, const float* q, int qn, long long qs, 
     case 16: LS_LAUNCH(M, 16); break; \
     default: LS_LAUNCH(M, 32); break; \
   }
-  if (mode == 0) { LS_LANES(0) } else if (mode == 1) { LS_LANES(1) } else { LS_LANES(2) }
+  if (mode == 0) { LS_LANES(0) } else if (mode == 1) { LS_LANES(1) } else if (mode == 2) { LS_LANES(2) } else { LS_LANES(3) }
 #undef LS_LANES
 #undef LS_LAUNCH
   LLM_CHECK_LAUNCH("linear_state");
@@ -600,17 +677,40 @@ extern "C" int llm_delta_gates(const float* a, int an, long long as, int aw, int
   return LLM_OK;
 }
 
+// x: float32 sums; columns x0.. (R0 of them) and x1.. (R1). wt0 [R0, C0], wt1 [R1, C1]: the maps transposed, in the engine's dtype.
+extern "C" int llm_channel_gates(const float* x, int xn, long long xs, int xw, int x0, int x1, int R0, int R1, const void* wt0, const void* wt1,
+                                 const float* bias0, const float* a_log, int C0, int C1, int per, float* out0, float* out1, int dtype,
+                                 int n_tokens, cudaStream_t stream) {
+  if (n_tokens == 0) return LLM_OK;
+  LLM_REQUIRE(n_tokens > 0 && x && xn >= 1 && wt0 && wt1 && bias0 && a_log && out0 && out1, "channel_gates: missing tensors");
+  LLM_REQUIRE(R0 > 0 && R1 > 0 && C0 > 0 && C1 > 0 && per > 0 && C0 % per == 0, "channel_gates: bad sizes");
+  LLM_REQUIRE(x0 >= 0 && x1 >= 0 && x0 + R0 <= xw && x1 + R1 <= xw, "channel_gates: columns outside the product");
+  LLM_REQUIRE(dtype == LLM_F32 || dtype == LLM_BF16, "channel_gates: unknown dtype %d", dtype);
+  ChannelGates p;
+  p.x0 = Sums{x, xn, (size_t)xs, xw, x0}; p.x1 = Sums{x, xn, (size_t)xs, xw, x1};
+  p.R0 = R0; p.R1 = R1; p.C0 = C0; p.C1 = C1; p.per = per; p.bias0 = bias0; p.a_log = a_log; p.out0 = out0; p.out1 = out1; p.n_tokens = n_tokens;
+  const size_t smem = ((size_t)max(R0, R1) * 8 + 4 * 32 * 8) * sizeof(float);
+  LLM_REQUIRE(smem <= 48 * 1024, "channel_gates: ranks of %d / %d exceed one block's shared memory", R0, R1);
+  dim3 grid(ceil_div(C0, 32) + ceil_div(C1, 32), ceil_div(n_tokens, 8));
+  LLM_REQUIRE(grid.y <= 65535, "channel_gates: too many tokens in one step (%d)", n_tokens);
+  if (dtype == LLM_F32) launch_kernel(channel_gates_kernel<float>, grid, 128, smem, stream, p, (const float*)wt0, (const float*)wt1);
+  else launch_kernel(channel_gates_kernel<bf16>, grid, 128, smem, stream, p, (const bf16*)wt0, (const bf16*)wt1);
+  LLM_CHECK_LAUNCH("channel_gates");
+  return LLM_OK;
+}
+
 extern "C" int llm_head_norm_gate(const float* o, const float* weight, int weight_per_head, const float* gate, int gn, long long gs, int gw,
-                                  int go, float eps, void* out, int dtype, int n_tokens, int H, int dv, cudaStream_t stream) {
+                                  int go, float eps, void* out, int dtype, int n_tokens, int H, int dv, int sigmoid, cudaStream_t stream) {
+  // sigmoid 1: the gate is sigmoid(sums) instead of silu(sums)
   if (n_tokens == 0) return LLM_OK;
   LLM_REQUIRE(n_tokens > 0 && H > 0 && dv > 0 && o && weight && out, "head_norm_gate: bad arguments");
   LLM_REQUIRE(gate == nullptr || (gn >= 1 && go >= 0 && go + H * dv <= gw), "head_norm_gate: gate columns outside the product");
   const Sums g{gate, gn, (size_t)gs, gw, go};
   const int blocks = ceil_div((long long)n_tokens * H, 4);
   if (dtype == LLM_F32)
-    launch_kernel(head_norm_gate_kernel<float>, blocks, 128, 0, stream, o, weight, weight_per_head, g, eps, (float*)out, n_tokens, H, dv);
+    launch_kernel(head_norm_gate_kernel<float>, blocks, 128, 0, stream, o, weight, weight_per_head, g, eps, (float*)out, n_tokens, H, dv, sigmoid);
   else if (dtype == LLM_BF16)
-    launch_kernel(head_norm_gate_kernel<bf16>, blocks, 128, 0, stream, o, weight, weight_per_head, g, eps, (bf16*)out, n_tokens, H, dv);
+    launch_kernel(head_norm_gate_kernel<bf16>, blocks, 128, 0, stream, o, weight, weight_per_head, g, eps, (bf16*)out, n_tokens, H, dv, sigmoid);
   else
     LLM_REQUIRE(false, "head_norm_gate: unknown dtype %d", dtype);
   LLM_CHECK_LAUNCH("head_norm_gate");

@@ -221,7 +221,7 @@ __global__ void __launch_bounds__(RM_THREADS)
 __global__ void __launch_bounds__(RM_THREADS)
     heads_product_mma_kernel(const bf16* __restrict__ a, long long lda, long long lda_h, const bf16* __restrict__ w, int T_, int N, int K,
                              bf16* __restrict__ out, long long ldo, long long ldo_h, const float* __restrict__ gate, int n_parts,
-                             size_t pstride, int gwidth, int g_off) {
+                             size_t pstride, int gwidth, int g_off, int g_head) {
   extern __shared__ __align__(16) uint8_t smem_raw[];
   bf16 (*a_s)[RM_ROWS][RM_LD] = reinterpret_cast<bf16 (*)[RM_ROWS][RM_LD]>(smem_raw);
   bf16 (*w_s)[RM_COLS][RM_LD] = reinterpret_cast<bf16 (*)[RM_COLS][RM_LD]>(smem_raw + (size_t)RM_STAGES * RM_ROWS * RM_LD * sizeof(bf16));
@@ -286,7 +286,7 @@ __global__ void __launch_bounds__(RM_THREADS)
         if (n >= N) continue;
         float v = acc[j][2 * half + el];
         if (gate) {
-          const size_t gi = (size_t)t * gwidth + g_off + (size_t)h * N + n;
+          const size_t gi = (size_t)t * gwidth + g_off + (g_head ? (size_t)h : (size_t)h * N + n);  // g_head: one gate a head
           float g = gate[gi];
           for (int q = 1; q < n_parts; ++q) g += gate[(size_t)q * pstride + gi];  // index order
           v *= 1.0f / (1.0f + expf(-g));
@@ -383,7 +383,7 @@ extern "C" int llm_heads_product_mma_supported(const void* a, long long lda, lon
 
 extern "C" int llm_heads_product_mma(const void* a, long long lda, long long lda_h, const void* w, void* out, long long ldo, long long ldo_h,
                                      int n_tokens, int H, int N, int K, const float* gate, int n_parts, long long pstride, int gwidth,
-                                     int g_off, cudaStream_t stream) {
+                                     int g_off, int g_head, cudaStream_t stream) {
   if (n_tokens == 0) return LLM_OK;
   LLM_REQUIRE(llm_heads_product_mma_supported(a, lda, lda_h, w, K), "heads_product_mma: operands must be 16-byte aligned with K and the strides multiples of 8");
   LLM_REQUIRE(n_tokens > 0 && H > 0 && N > 0 && H <= 65535 && ceil_div(n_tokens, RM_ROWS) <= 65535, "heads_product_mma: bad sizes");
@@ -395,7 +395,7 @@ extern "C" int llm_heads_product_mma(const void* a, long long lda, long long lda
   }
   dim3 grid(ceil_div(N, RM_COLS), ceil_div(n_tokens, RM_ROWS), H);
   launch_kernel(heads_product_mma_kernel, grid, RM_THREADS, RM_SMEM, stream, (const bf16*)a, lda, lda_h, (const bf16*)w, n_tokens, N, K,
-                (bf16*)out, ldo, ldo_h, gate, n_parts, (size_t)pstride, gwidth, g_off);
+                (bf16*)out, ldo, ldo_h, gate, n_parts, (size_t)pstride, gwidth, g_off, g_head);
   LLM_CHECK_LAUNCH("heads_product_mma");
   return LLM_OK;
 }

@@ -172,7 +172,7 @@ class Engine:
             num_slots = num_slots or self._default_slots
             H = host_module()
             self.cm = H.CacheManager(block_size, [H.GroupSpec(num_blocks, w) for w in model.windows], num_slots)
-            for c in model.caches:  # drop the old pool before the new one is made
+            for c in (*model.caches, model.embedding_cache):  # drop the old pool before the new one is made
                 c.k = c.v = None
                 c.states = {}
             model.allocate_cache([num_blocks] * len(model.windows), num_slots)

@@ -13,7 +13,7 @@ from typing import List, Optional, Sequence
 import torch
 
 from ..cache.storage import allocate_run_caches, bytes_per_token, plan_groups
-from ..parts.base import BuildEnv, LayerCache, Residual
+from ..parts.base import BuildEnv, LayerCache, Residual, StateNeed
 from ..parts.registry import build_part
 from ..parts.spec import ModelSpec
 from ..weights.loader import Checkpoint, load_tensors
@@ -40,15 +40,20 @@ class Model:
         self.run_needs: List[Sequence[object]] = [
             () if run.cache_from is not None else tuple(self.blocks[run.layer].cache_needs()) for run in spec.order]
         self.windows, self.run_group = plan_groups(self.run_needs)
+        # what the embedding keeps per request (state alone: it has no keys and values)
+        self.embedding_needs: Sequence[object] = tuple(self.embedding.cache_needs())
+        if any(not isinstance(n, StateNeed) for n in self.embedding_needs):
+            raise ValueError("an embedding may keep state, but no keys and values")
         # where the scheduler may cut a prompt: the least common multiple of what the layers ask for
         self.portion_multiple = 1
-        for needs in self.run_needs:
+        for needs in (*self.run_needs, self.embedding_needs):
             for need in needs:
                 m = int(getattr(need, "portion_multiple", 1))
                 if m < 1:
                     raise ValueError(f"cache need {need!r}: portion_multiple must be >= 1")
                 self.portion_multiple = math.lcm(self.portion_multiple, m)
         self.caches: List[LayerCache] = [LayerCache() for _ in range(n_runs)]
+        self.embedding_cache = LayerCache()
         self.weight_bytes = 0
         # for looking at a model layer by layer: called as after_run(run index, float32 stream [tokens, hidden]) behind every
         # run of a layer, with everything that the run left pending added (the same sum the next norm would have made)
@@ -71,6 +76,8 @@ class Model:
     def allocate_cache(self, group_pages: Sequence[int], num_slots: int) -> None:
         own = allocate_run_caches(self.run_needs, self.run_group, group_pages, self.windows, self.env.page_size,
                                   num_slots, self.env.dtype, self.env.device)
+        self.embedding_cache = allocate_run_caches([self.embedding_needs], [None], group_pages, self.windows, self.env.page_size,
+                                                   num_slots, self.env.dtype, self.env.device)[0]
         for r, run in enumerate(self.spec.order):
             if run.cache_from is None:
                 self.caches[r] = own[r]
@@ -81,7 +88,7 @@ class Model:
 
     def reset_slot(self, slot: int) -> None:
         """A request starts in this slot: its fixed-size state begins at zero."""
-        for c in self.caches:
+        for c in (*self.caches, self.embedding_cache):
             if c.writes:
                 for t in c.states.values():
                     t[slot].zero_()
@@ -112,6 +119,7 @@ class Model:
     def forward(self, ctx) -> torch.Tensor:
         order = self.spec.order
         ctx.stream_sumsq = ctx.stream_prescaled = None
+        ctx.embedding_cache = self.embedding_cache
         # who reads the residual stream next: a part that writes it may leave that norm's input prepared
         ctx.next_norm = self.blocks[order[0].layer].first_norm() if order else self.final_norm
         res = Residual(self.embedding.forward(ctx))

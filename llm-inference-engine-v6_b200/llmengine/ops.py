@@ -180,6 +180,23 @@ class CudaOps:
                                   c_longlong(ld_scaled), c_float(scale), _stream()), lib)
         return out
 
+    def embed_pairs(self, table: torch.Tensor, pairs: torch.Tensor, buckets: int, mul_prev: int, mul_cur: int, scale: float,
+                    previous: torch.Tensor, batch, out: torch.Tensor) -> torch.Tensor:
+        """out[t] (float32) = table[id] * scale + pairs[row], row = (id of the request's token before t * mul_prev + id * mul_cur)
+        mod buckets, or `buckets` at position 0. previous (int32 [slots, 1]): the token before a portion's first one, by the
+        request's slot; afterwards the portion's last token."""
+        _need(table, "embed_pairs.table"); _need(pairs, "embed_pairs.pairs", table.dtype); _need(out, "embed_pairs.out", torch.float32)
+        _need(previous, "embed_pairs.previous", torch.int32)
+        n, dim = batch.n_tokens, out.shape[1]
+        assert table.is_contiguous() and pairs.is_contiguous() and out.is_contiguous() and previous.is_contiguous() and out.shape[0] >= n
+        assert table.shape[1] == dim and tuple(pairs.shape) == (buckets + 1, dim) and previous.numel() == previous.shape[0]
+        lib = self.lib()
+        self._check(lib.llm_embed_pairs(_ptr(table), _ptr(pairs), c_int(dtype_code(table.dtype)), c_int(buckets), c_longlong(mul_prev),
+                                        c_longlong(mul_cur), c_float(scale), _ptr(batch.token_ids), _ptr(batch.positions), _ptr(batch.token_seq),
+                                        _ptr(batch.seq_qoff), _ptr(batch.seq_ntok), _ptr(batch.seq_slot), _ptr(previous), _ptr(out), c_int(n),
+                                        c_int(dim), c_int(table.shape[0]), _stream()), lib)
+        return out
+
     def rmsnorm(self, h: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor,
                 delta: Optional[torch.Tensor] = None, rows: Optional[torch.Tensor] = None,
                 n_rows: Optional[int] = None, write_back: bool = True, center: bool = False) -> torch.Tensor:
@@ -335,11 +352,11 @@ class CudaOps:
         return out
 
     def gemm_heads(self, a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, gate: Optional[torch.Tensor] = None,
-                   gate_off: int = 0) -> bool:
+                   gate_off: int = 0, gate_per_head: bool = False) -> bool:
         """out[:, h, :] = a[:, h, :] @ w[h].T for all heads in one tensor-core launch (a [n, H, K], w [H, N, K], out
         [n, H, N] bfloat16; views whose last dimension is contiguous); with gate (float32 partial sums [p, n, width]),
-        times sigmoid(sum_p gate[p, t, gate_off + h*N + j]). False, with nothing done, when the operands are not what
-        that kernel takes (the caller then uses heads_product)."""
+        times sigmoid(sum_p gate[p, t, gate_off + h*N + j]), or with gate_per_head one gate a head at column gate_off + h. False,
+        with nothing done, when the operands are not what that kernel takes (the caller then uses heads_product)."""
         if a.dtype != torch.bfloat16 or not self.tensor_cores or a.stride(2) != 1 or out.stride(2) != 1:
             return False
         n, H, K = a.shape
@@ -351,11 +368,11 @@ class CudaOps:
         gargs = (c_void_p(0), c_int(0), c_longlong(0), c_int(0), c_int(0))
         if gate is not None:
             _need(gate, "gemm_heads.gate", torch.float32)
-            assert gate.is_contiguous() and gate.dim() == 3 and gate.shape[1] >= n and gate_off + H * N <= gate.shape[2]
+            assert gate.is_contiguous() and gate.dim() == 3 and gate.shape[1] >= n and gate_off + H * (1 if gate_per_head else N) <= gate.shape[2]
             gargs = (_ptr(gate), c_int(gate.shape[0]), c_longlong(gate.stride(0)), c_int(gate.shape[2]), c_int(gate_off))
         self._check(lib.llm_heads_product_mma(_ptr(a), c_longlong(a.stride(0)), c_longlong(a.stride(1)), _ptr(w), _ptr(out),
                                               c_longlong(out.stride(0)), c_longlong(out.stride(1)), c_int(n), c_int(H), c_int(N), c_int(K),
-                                              *gargs, _stream()), lib)
+                                              *gargs, c_int(1 if gate_per_head else 0), _stream()), lib)
         return True
 
     def gemm_partials(self, a: torch.Tensor, w: torch.Tensor, ws, tag: str) -> torch.Tensor:
@@ -820,17 +837,20 @@ class CudaOps:
 
     # ------------------------------------------------------------------ latent attention
     def latent_prep(self, parts: torch.Tensor, q_off: int, q_rank: int, kv_off: int, kv_rank: int, rot_dim: int, rot_dims: int,
-                    wq: torch.Tensor, wkv: torch.Tensor, eps: float, cos: Optional[torch.Tensor], sin: Optional[torch.Tensor],
+                    wq: torch.Tensor, wkv: Optional[torch.Tensor], eps: float, cos: Optional[torch.Tensor], sin: Optional[torch.Tensor],
                     batch, block_table: torch.Tensor, cq: torch.Tensor, cache: Optional[torch.Tensor]) -> None:
         """From the float32 partial sums parts [p, n, width] of the mixer's first product: cq [n, q_rank] = the RMS-normed
         query latent (weight wq); the cache row [c | kr] of every token, c = the RMS-normed first kv_rank numbers of the
         key/value columns (weight wkv), kr = the next rot_dim with the first rot_dims rotated by cos/sin [positions, rot_dims/2].
-        cache [pages, 1, page_size, kv_rank + rot_dim], or None for a run that writes none."""
+        cache [pages, 1, page_size, kv_rank + rot_dim], or None for a run that writes none. kv_rank 0: the product holds no
+        key/value columns (the layer reads another layer's latents), wkv and cache are None."""
         _need(parts, "latent_prep.parts", torch.float32); _need(cq, "latent_prep.cq"); _need(block_table, "latent_prep.block_table", torch.int32)
-        _need(wq, "latent_prep.wq", torch.float32); _need(wkv, "latent_prep.wkv", torch.float32)
+        _need(wq, "latent_prep.wq", torch.float32)
+        if kv_rank:
+            _need(wkv, "latent_prep.wkv", torch.float32)
         n = batch.n_tokens
         assert parts.is_contiguous() and parts.dim() == 3 and parts.shape[1] >= n and block_table.is_contiguous()
-        assert wq.numel() == q_rank and wkv.numel() == kv_rank and cq.shape[0] >= n and cq.shape[1] == q_rank
+        assert wq.numel() == q_rank and (wkv.numel() if kv_rank else 0) == kv_rank and cq.shape[0] >= n and cq.shape[1] == q_rank
         page = 1
         if cache is not None:
             _need(cache, "latent_prep.cache", cq.dtype)
@@ -848,9 +868,10 @@ class CudaOps:
                                         _stream()), lib)
 
     def heads_product(self, a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, gate: Optional[torch.Tensor] = None,
-                      gate_off: int = 0) -> torch.Tensor:
+                      gate_off: int = 0, gate_per_head: bool = False) -> torch.Tensor:
         """out[t, h, :] = w[h] a[t, h, :] for a [n, H, K], w [H, N, K], out [n, H, N] (views whose last dimension is
-        contiguous); with gate (float32 partial sums [p, n, width]), times sigmoid(sum_p gate[p, t, gate_off + h*N + j])."""
+        contiguous); with gate (float32 partial sums [p, n, width]), times sigmoid(sum_p gate[p, t, gate_off + h*N + j]), or with
+        gate_per_head one gate a head at column gate_off + h."""
         _need(a, "heads_product.a"); _need(w, "heads_product.w", a.dtype); _need(out, "heads_product.out", a.dtype)
         n, H, K = a.shape
         N = w.shape[1]
@@ -858,12 +879,12 @@ class CudaOps:
         gargs = (c_void_p(0), c_int(0), c_longlong(0), c_int(0), c_int(0))
         if gate is not None:
             _need(gate, "heads_product.gate", torch.float32)
-            assert gate.is_contiguous() and gate.dim() == 3 and gate.shape[1] >= n and gate_off + H * N <= gate.shape[2]
+            assert gate.is_contiguous() and gate.dim() == 3 and gate.shape[1] >= n and gate_off + H * (1 if gate_per_head else N) <= gate.shape[2]
             gargs = (_ptr(gate), c_int(gate.shape[0]), c_longlong(gate.stride(0)), c_int(gate.shape[2]), c_int(gate_off))
         lib = self.lib()
         self._check(lib.llm_heads_product(_ptr(a), c_longlong(a.stride(0)), c_longlong(a.stride(1)), _ptr(w), c_longlong(K), _ptr(out),
                                           c_longlong(out.stride(0)), c_longlong(out.stride(1)), c_int(n), c_int(H), c_int(N), c_int(K),
-                                          *gargs, c_int(dtype_code(a.dtype)), _stream()), lib)
+                                          *gargs, c_int(1 if gate_per_head else 0), c_int(dtype_code(a.dtype)), _stream()), lib)
         return out
 
     def latent_query(self, q: torch.Tensor, wkt: Optional[torch.Tensor], ql: torch.Tensor, heads: int, dim: int, rot_dim: int,
@@ -885,20 +906,25 @@ class CudaOps:
         return ql
 
     def latent_attention(self, ql: torch.Tensor, cache: torch.Tensor, batch, block_table: torch.Tensor, out: torch.Tensor,
-                         kv_rank: int, scale: float, window: int = 0) -> torch.Tensor:
+                         kv_rank: int, scale: float, window: int = 0, sink: Optional[torch.Tensor] = None) -> torch.Tensor:
         """Causal softmax attention of every token of the step over the cached rows lo..pos of its request: ql [n, H, Dk]
-        against cache [pages, 1, page_size, Dk]; the values are the first kv_rank numbers of the rows; out [n, H, kv_rank]."""
+        against cache [pages, 1, page_size, Dk]; the values are the first kv_rank numbers of the rows; out [n, H, kv_rank].
+        sink (float32 [H], optional): exp(sink[head]) is one more term of the softmax's denominator."""
         _need(ql, "latent_attention.ql"); _need(cache, "latent_attention.cache", ql.dtype); _need(out, "latent_attention.out", ql.dtype)
         _need(block_table, "latent_attention.block_table", torch.int32)
         n, H, Dk = ql.shape
         assert ql.is_contiguous() and out.is_contiguous() and cache.is_contiguous() and block_table.is_contiguous()
         assert cache.shape[1] == 1 and cache.shape[3] == Dk and out.shape == (n, H, kv_rank) and n >= batch.n_tokens
+        if sink is not None:
+            _need(sink, "latent_attention.sink", torch.float32)
+            assert sink.numel() == H and sink.is_contiguous()
         if ql.dtype == torch.bfloat16 and self.tensor_cores and self.latent_tensor_cores:
             lib = self.lib("tensorcore")
             if lib.llm_latent_attention_mma_supported(c_int(H), c_int(kv_rank), c_int(Dk - kv_rank)):
                 n_splits, split_keys, scratch = 1, 256, None
                 if batch.max_new_tokens == 1 and batch.n_tokens == batch.n_seqs:
-                    n_splits, split_keys = self._latent_split_policy(batch.n_seqs * -(-H // 32), batch.max_seq_len)
+                    reach = min(batch.max_seq_len, window + 63) if window > 0 else batch.max_seq_len  # splits begin at the window's tile
+                    n_splits, split_keys = self._latent_split_policy(batch.n_seqs * -(-H // 32), reach)
                 if n_splits > 1:
                     floats = int(lib.llm_latent_attention_scratch_floats(c_int(batch.n_tokens), c_int(H), c_int(kv_rank), c_int(n_splits)))
                     scratch = batch.ws.get("latent.splits", (floats,), torch.float32)
@@ -906,7 +932,7 @@ class CudaOps:
                     _ptr(ql), _ptr(cache), _ptr(batch.seq_start), _ptr(batch.seq_ntok), _ptr(batch.seq_qoff), _ptr(block_table),
                     c_int(block_table.shape[1]), _ptr(out), c_int(batch.n_seqs), c_int(batch.n_tokens), c_int(batch.max_new_tokens),
                     c_int(H), c_int(kv_rank), c_int(Dk - kv_rank), c_int(cache.shape[2]), c_float(scale), c_int(window),
-                    c_int(n_splits), c_int(split_keys), _ptr(scratch), _stream()), lib)
+                    c_int(n_splits), c_int(split_keys), _ptr(scratch), _ptr(sink), _stream()), lib)
                 if n_splits > 1:
                     self.launches += 1  # the kernel that merges the splits
                 return out
@@ -914,7 +940,7 @@ class CudaOps:
         self._check(lib.llm_latent_attention_simt(_ptr(ql), _ptr(cache), c_int(dtype_code(ql.dtype)), _ptr(batch.positions),
                                                   _ptr(batch.token_seq), _ptr(block_table), c_int(block_table.shape[1]), _ptr(out),
                                                   c_int(batch.n_tokens), c_int(H), c_int(kv_rank), c_int(Dk - kv_rank),
-                                                  c_int(cache.shape[2]), c_float(scale), c_int(window), _stream()), lib)
+                                                  c_int(cache.shape[2]), c_float(scale), c_int(window), _ptr(sink), _stream()), lib)
         return out
 
     LATENT_TARGET_CTAS = 296  # two CTAs of the latent attention kernel on each of the 148 SMs
@@ -1109,25 +1135,31 @@ class CudaOps:
                  k_norm: Optional[torch.Tensor], eps: float, cos: Optional[torch.Tensor], sin: Optional[torch.Tensor], batch,
                  block_table: torch.Tensor, q_out: torch.Tensor, kcache: Optional[torch.Tensor], vcache: Optional[torch.Tensor],
                  mix_role: int = 0, mix_weight: Optional[torch.Tensor] = None, v_first: Optional[torch.Tensor] = None,
-                 norm_wide: bool = False) -> None:
+                 norm_wide: bool = False, bias: Optional[torch.Tensor] = None, neighbours: bool = False, unit_rms: bool = False,
+                 keys_as_values: bool = False) -> None:
         """From the float32 sums `parts` [p, n, width] of a product whose columns begin with [q: heads * dk | k: kv_heads * dk |
         v: kv_heads * dv] (kv_heads 0: queries alone, nothing to write): RMS norm of every query and key head with the weights
         q_norm / k_norm [dk] (None: no norm), or with norm_wide ONE RMS norm over all query heads' numbers together with q_norm
         [heads * dk] and one over all key heads' with k_norm [kv_heads * dk]; rotation
         of the first 2 * cos.shape[1] numbers of each head (half-split pairs) at the token's position, q into q_out
         [n, heads * dk], k and v into the token's page of kcache [pages, kv_heads, page, dk] / vcache [.., dv] (None: no write).
+        bias (float32 [(heads + kv_heads) * dk]) is added to the q and k columns first; neighbours: the rotation's pairs are (2i, 2i + 1);
+        unit_rms: every head is divided by its root mean square after the rotation; keys_as_values: the product has no v columns, the
+        values are its k columns (with their bias, before norm and rotation; dv == dk).
         mix_role 1: the values are also left in v_first (float32 [n, kv_heads * dv]); 2: v <- (1 - m) v + m v_first before
         the write, m = mix_weight (a float32 scalar on the device)."""
         _need(parts, "qkv_prep.parts", torch.float32); _need(q_out, "qkv_prep.q")
         assert parts.dim() == 3 and parts.is_contiguous()
         n = batch.n_tokens
         rot_dims = 0 if cos is None else 2 * cos.shape[1]
-        for t, name in ((q_norm, "q_norm"), (k_norm, "k_norm"), (cos, "cos"), (sin, "sin"), (mix_weight, "mix_weight"), (v_first, "v_first")):
+        for t, name in ((q_norm, "q_norm"), (k_norm, "k_norm"), (cos, "cos"), (sin, "sin"), (mix_weight, "mix_weight"), (v_first, "v_first"),
+                        (bias, "bias")):
             if t is not None:
                 _need(t, "qkv_prep." + name, torch.float32)
                 assert t.is_contiguous()
         wide = (heads, kv_heads) if norm_wide else (1, 1)
         assert (q_norm is None or q_norm.numel() == wide[0] * dk) and (k_norm is None or kv_heads == 0 or k_norm.numel() == wide[1] * dk)
+        assert bias is None or bias.numel() == (heads + kv_heads) * dk
         page = 1
         if kcache is not None:
             _need(kcache, "qkv_prep.kcache", q_out.dtype); _need(vcache, "qkv_prep.vcache", q_out.dtype)
@@ -1142,7 +1174,8 @@ class CudaOps:
                                      _ptr(cos), _ptr(sin), _ptr(batch.positions), _ptr(batch.token_seq), _ptr(block_table),
                                      c_int(block_table.shape[1]), _ptr(q_out), c_longlong(q_out.stride(0)), _ptr(kcache), _ptr(vcache),
                                      c_int(page), c_int(mix_role), _ptr(mix_weight), _ptr(v_first), c_int(dtype_code(q_out.dtype)),
-                                     c_int(n), c_int(1 if norm_wide else 0), _stream()), lib)
+                                     c_int(n), c_int(1 if norm_wide else 0), _ptr(bias), c_int(1 if neighbours else 0),
+                                     c_int(1 if unit_rms else 0), c_int(1 if keys_as_values else 0), _stream()), lib)
 
     def gated_attention(self, q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor, batch, block_table: torch.Tensor,
                         out: torch.Tensor, nq: int, nkv: int, dk: int, dv: int, scale: float, window: int = 0, chunk: int = 0,
@@ -1171,8 +1204,9 @@ class CudaOps:
             if lib.llm_gated_attention_mma_supported(c_int(nq), c_int(nkv), c_int(dk), c_int(dv), c_longlong(q.stride(0)), c_longlong(out.stride(0))):
                 n_splits, split_keys, scratch = 1, 256, None
                 if batch.max_new_tokens == 1 and batch.n_tokens == batch.n_seqs and dk == dv:
-                    # single decoded tokens: the keys a token may see (its chunk at most) in pieces side by side
-                    reach = min(batch.max_seq_len, chunk) if chunk > 0 else batch.max_seq_len
+                    # single decoded tokens: the keys a token may see (its chunk or window at most) in pieces side by side; a
+                    # window's pieces are counted from its first key's tile of 64
+                    reach = min(batch.max_seq_len, chunk) if chunk > 0 else min(batch.max_seq_len, window + 63) if window > 0 else batch.max_seq_len
                     n_splits, split_keys = self._split_policy(batch.n_seqs * nkv, reach, dk)
                     if n_splits > 1:
                         floats = int(lib.llm_attention_mma_scratch_floats(c_int(batch.n_tokens), c_int(nq), c_int(dv), c_int(n_splits)))
@@ -1328,7 +1362,7 @@ class CudaOps:
         return out
 
     # ------------------------------------------------------------------ mixers with a matrix of state per head
-    LINEAR_STATE_RULES = {"decay_write_read": 0, "bonus_read_decay_write": 1, "delta": 2}
+    LINEAR_STATE_RULES = {"decay_write_read": 0, "bonus_read_decay_write": 1, "delta": 2, "channel_delta": 3}
 
     def linear_state_shape(self, heads: int, dk: int, dv: int):
         """Shape of the float32 state that linear_state keeps per request (its layout is the kernel's own)."""
@@ -1348,11 +1382,12 @@ class CudaOps:
 
     def linear_state(self, rule: str, q, q_off: int, k, k_off: int, v, v_off: int, decay: torch.Tensor, decay_off: int,
                      bonus: Optional[torch.Tensor], state: torch.Tensor, batch, out: torch.Tensor, heads: int, kv_heads: int, dk: int,
-                     dv: int, q_scale: float = 1.0, unit_eps: float = -1.0, decay_const: bool = False) -> torch.Tensor:
+                     dv: int, q_scale: float = 1.0, unit_eps: float = -1.0, decay_const: bool = False, beta=None, beta_off: int = 0) -> torch.Tensor:
         """Token after token of every request, per head a matrix S [dk, dv] (float32, in the request's slot of `state`):
         "decay_write_read": S <- diag(a) S + k v^T, o = S^T q; "bonus_read_decay_write": o = (S + diag(bonus) k v^T)^T q, then
         S <- diag(a) S + k v^T; "delta": S <- g S, w = beta (v - S^T k), S <- S + k w^T, o = S^T q with q and k made unit vectors
-        per head first (x / sqrt(sum x^2 + unit_eps); unit_eps < 0: as they are). q is multiplied by q_scale. q, k, v: float32 sums
+        per head first (x / sqrt(sum x^2 + unit_eps); unit_eps < 0: as they are); "channel_delta": the same with S <- diag(a) S for its
+        first step and beta = the sigmoid of the float32 sums `beta` at column beta_off + head. q is multiplied by q_scale. q, k, v: float32 sums
         ([parts, n, width] or [n, width]) read at column offsets, q and k with kv_heads heads of dk (head h reads head
         h // (heads / kv_heads)), v with heads of dv. decay: float32 rows; at decay_off a number per (head, key channel), or for
         "delta" [g: heads | beta: heads]; with decay_const a single row that holds for every token (decays that are constants
@@ -1363,9 +1398,11 @@ class CudaOps:
         if bonus is not None:
             _need(bonus, "linear_state.bonus", torch.float32)
             assert bonus.is_contiguous() and bonus.numel() == heads * dk
+        assert (beta is not None) == (rule == "channel_delta")
+        b_args = self._sums(beta, beta_off, "linear_state.beta") if beta is not None else [c_void_p(0), c_int(0), c_longlong(0), c_int(0), c_int(0)]
         lib = self.lib()
         self._check(lib.llm_linear_state(c_int(self.LINEAR_STATE_RULES[rule]), *self._sums(q, q_off, "linear_state.q"),
-                                         *self._sums(k, k_off, "linear_state.k"), *self._sums(v, v_off, "linear_state.v"), _ptr(decay),
+                                         *self._sums(k, k_off, "linear_state.k"), *self._sums(v, v_off, "linear_state.v"), *b_args, _ptr(decay),
                                          c_int(decay.shape[1]), c_int(decay_off), _ptr(bonus), _ptr(state), _ptr(batch.seq_qoff),
                                          _ptr(batch.seq_ntok), _ptr(batch.seq_slot), _ptr(out), c_int(batch.n_tokens), c_int(batch.n_seqs), c_int(heads),
                                          c_int(kv_heads), c_int(dk), c_int(dv), c_float(q_scale), c_float(unit_eps), c_int(1 if decay_const else 0),
@@ -1417,17 +1454,40 @@ class CudaOps:
                                         _ptr(dt_bias), _ptr(out), c_int(n_tokens), c_int(H), _stream()), lib)
         return out
 
+    def channel_gates(self, sums, decay_col: int, decay_rank: int, gate_col: int, gate_rank: int, decay_t: torch.Tensor, gate_t: torch.Tensor,
+                      dt_bias: torch.Tensor, a_log: torch.Tensor, decay: torch.Tensor, gate: torch.Tensor, n_tokens: int) -> None:
+        """Two low-rank maps of the float32 `sums` [parts, n, width] in one launch: decay[t, c] = exp(-exp(a_log[c // per]) *
+        softplus(dt_bias[c] + sum_r decay_t[r, c] * sums[t, decay_col + r])) with per = channels / len(a_log), and
+        gate[t, c] = sum_r gate_t[r, c] * sums[t, gate_col + r]. decay_t, gate_t [rank, channels]: the maps stored transposed;
+        decay, gate: float32 [n, channels]."""
+        for t, name in ((dt_bias, "dt_bias"), (a_log, "a_log"), (decay, "decay"), (gate, "gate")):
+            _need(t, "channel_gates." + name, torch.float32)
+            assert t.is_contiguous()
+        _need(decay_t, "channel_gates.decay_t"); _need(gate_t, "channel_gates.gate_t", decay_t.dtype)
+        C0, C1 = decay_t.shape[1], gate_t.shape[1]
+        assert decay_t.is_contiguous() and gate_t.is_contiguous() and decay_t.shape[0] == decay_rank and gate_t.shape[0] == gate_rank
+        assert dt_bias.numel() == C0 and C0 % a_log.numel() == 0 and decay.shape[1] == C0 and gate.shape[1] == C1
+        assert decay.shape[0] >= n_tokens and gate.shape[0] >= n_tokens
+        p, parts, stride, width, _ = self._sums(sums, 0, "channel_gates.sums")
+        lib = self.lib()
+        self._check(lib.llm_channel_gates(p, parts, stride, width, c_int(decay_col), c_int(gate_col), c_int(decay_rank), c_int(gate_rank),
+                                          _ptr(decay_t), _ptr(gate_t), _ptr(dt_bias), _ptr(a_log), c_int(C0), c_int(C1),
+                                          c_int(C0 // a_log.numel()), _ptr(decay), _ptr(gate), c_int(dtype_code(decay_t.dtype)), c_int(n_tokens),
+                                          _stream()), lib)
+
     def head_norm_gate(self, o: torch.Tensor, weight: torch.Tensor, gate, gate_off: int, eps: float, out: torch.Tensor, n_tokens: int,
-                       heads: int, dv: int) -> torch.Tensor:
-        """out[t, h] = o[t, h] / sqrt(mean(o[t, h]^2) + eps) * weight * silu(gate[t, h]) per head of dv numbers; o float32
-        [n, heads * dv]; weight float32 [dv] (one for all heads) or [heads * dv]; gate: float32 sums read at gate_off (None: no gate)."""
+                       heads: int, dv: int, act: str = "silu") -> torch.Tensor:
+        """out[t, h] = o[t, h] / sqrt(mean(o[t, h]^2) + eps) * weight * act(gate[t, h]) per head of dv numbers, act "silu" or "sigmoid";
+        o float32 [n, heads * dv]; weight float32 [dv] (one for all heads) or [heads * dv]; gate: float32 sums read at gate_off (None:
+        no gate)."""
         _need(o, "head_norm_gate.o", torch.float32); _need(weight, "head_norm_gate.weight", torch.float32); _need(out, "head_norm_gate.out")
         assert o.is_contiguous() and out.is_contiguous() and o.shape[1] == heads * dv and out.shape[1] == heads * dv
         assert weight.numel() in (dv, heads * dv) and weight.is_contiguous()
         g = self._sums(gate, gate_off, "head_norm_gate.gate") if gate is not None else [c_void_p(0), c_int(0), c_longlong(0), c_int(0), c_int(0)]
         lib = self.lib()
         self._check(lib.llm_head_norm_gate(_ptr(o), _ptr(weight), c_int(1 if (weight.numel() == heads * dv and heads > 1) else 0), *g, c_float(eps),
-                                           _ptr(out), c_int(dtype_code(out.dtype)), c_int(n_tokens), c_int(heads), c_int(dv), _stream()), lib)
+                                           _ptr(out), c_int(dtype_code(out.dtype)), c_int(n_tokens), c_int(heads), c_int(dv),
+                                           c_int({"silu": 0, "sigmoid": 1}[act]), _stream()), lib)
         return out
 
     # ------------------------------------------------------------------ sampling

@@ -147,6 +147,11 @@ class Part:
 class Embedding(Part):
     category = "embedding"
 
+    def cache_needs(self) -> Sequence[object]:
+        """StateNeed objects: what the embedding keeps per request between steps (the previous token, say). The model allocates
+        them as it does for a layer and hands them over in ctx.embedding_cache."""
+        return ()
+
     def forward(self, ctx) -> torch.Tensor:
         """The float32 residual stream [tokens, hidden] of the step's tokens (ctx.token_ids). It may
         leave ctx.stream_sumsq: float32 [tokens, parts], the parts of every row's sum of squares
@@ -155,7 +160,7 @@ class Embedding(Part):
 
     def lookup(self, ctx, out: torch.Tensor) -> torch.Tensor:
         """The same rows once more into `out` (float32 [tokens, hidden]), for a model whose layer order adds the
-        embedding's output to the stream again (LayerRun.add_embedding)."""
+        embedding's output to the stream again (LayerRun.add_embedding). Called right behind forward, before any layer has run."""
         raise NotImplementedError
 
 

@@ -12,7 +12,7 @@ from typing import List
 
 import torch
 
-from .base import Embedding, Head, NormalizedRows
+from .base import Embedding, Head, NormalizedRows, StateNeed
 from .registry import build_part, part_class, register_part
 from .spec import EmbeddingSpec, HeadSpec, TensorNeed
 
@@ -89,6 +89,39 @@ class NormedTokenLookup(TokenLookup):
         return self.norm.run(raw, ctx, None, ctx.n_tokens, out=out)
 
 
+class PairLookup(TokenLookup):
+    """The table row of each token id times `scale`, plus a row of a second table chosen by the token and the one before it
+    (EmbeddingSpec "lookup_pairs"). One kernel: a portion's first token finds its predecessor in the request's slot, which afterwards
+    holds the portion's last token; position 0 has none and takes the row behind the buckets."""
+
+    def __init__(self, spec: EmbeddingSpec, env):
+        super().__init__(spec, env)
+        if not spec.pair_weight or spec.pair_buckets < 1 or min(spec.pair_mul_prev, spec.pair_mul_cur) < 0:
+            raise ValueError("embedding 'lookup_pairs' needs the pair table, at least one bucket and multipliers that are not negative")
+        self.pairs = None
+
+    @staticmethod
+    def tensor_needs(spec: EmbeddingSpec) -> List[TensorNeed]:
+        return TokenLookup.tensor_needs(spec) + [TensorNeed(spec.pair_weight, (spec.pair_buckets + 1, spec.dim), "compute")]
+
+    def cache_needs(self):
+        return (StateNeed("embedding.previous", (1,), torch.int32),)
+
+    def load(self, tensors) -> None:
+        super().load(tensors)
+        self.pairs = tensors[self.spec.pair_weight]
+
+    def forward(self, ctx) -> torch.Tensor:
+        s = self.spec
+        h = ctx.ws.get("model.residual", (ctx.n_tokens, s.dim), torch.float32)
+        return self.env.ops.embed_pairs(self.table, self.pairs, s.pair_buckets, s.pair_mul_prev, s.pair_mul_cur, float(s.scale),
+                                        ctx.embedding_cache.states["embedding.previous"], ctx, h)
+
+    def lookup(self, ctx, out: torch.Tensor) -> torch.Tensor:
+        # the slot has moved on to the portion's last token: the rows are taken from the stream, which nobody has written yet
+        return out.copy_(ctx.ws.get("model.residual", (ctx.n_tokens, self.spec.dim), torch.float32))
+
+
 class LinearHead(Head):
     def __init__(self, spec: HeadSpec, env):
         super().__init__(spec, env)
@@ -128,4 +161,5 @@ class LinearHead(Head):
 
 register_part("embedding", "lookup", TokenLookup)
 register_part("embedding", "lookup_normed", NormedTokenLookup)
+register_part("embedding", "lookup_pairs", PairLookup)
 register_part("head", "linear", LinearHead)

@@ -8,6 +8,9 @@ With h the mixer's input, per token at position p:
     score_a(i, j) = (q_a(i) . k_b(j)) * scale,  b = a // (H / G),  j <= i in the same chunk (and inside the window)
     p_a(i, j) = exp(score) / (sum_j exp(score) + exp(sink_a))   the sink only enlarges the denominator
     out = Wo ((heads' results side by side) * sigmoid(g))       g: a gate a number of the result, or (gate_per_head) one a head
+With q_bias and k_bias the projections of queries and keys have biases; rot_pairs "neighbours" turns the numbers 2i and 2i + 1 of a
+head together instead of i and i + dims / 2; with unit_rms every query and key head is divided by its root mean square behind the
+rotation (no weight); with keys_as_values there is no Wv: v = k as the projection gives it, before norms and rotation.
 With norm_scope "projection" the two norms are over all of q and all of k at once (weights of the projections' sizes). A layer
 without keys and values of its own (own_kv False) forms queries only and reads the cache of the run its LayerRun names.
 Norms, rotation, scores, softmax and the gate are float32 in both engine precisions. v_first are the values that the
@@ -44,6 +47,14 @@ class GatedAttention(Mixer):
             raise ValueError("gated attention: a layer that borrows keys and values has no key norm and mixes no values")
         if spec.value_mix not in (None, "first", "mix") or (spec.value_mix == "mix" and not spec.value_mix_weight):
             raise ValueError("gated attention: value_mix is None, 'first' or 'mix' (with the name of its weight)")
+        if spec.rot_pairs not in ("half", "neighbours"):
+            raise ValueError("gated attention: rot_pairs is 'half' or 'neighbours'")
+        if spec.unit_rms and (spec.q_norm or spec.k_norm):
+            raise ValueError("gated attention: unit_rms takes the place of the norms before the rotation")
+        if spec.keys_as_values and (spec.value_dim != spec.head_dim or spec.value_mix is not None or not spec.own_kv):
+            raise ValueError("gated attention: keys_as_values needs values of the keys' size, keys of the layer's own and no value mixing")
+        if (spec.q_bias or spec.k_bias or spec.unit_rms or spec.rot_pairs != "half") and spec.norm_scope != "head":
+            raise ValueError("gated attention: biases, unit_rms and neighbouring pairs go with norms a head")
         self.position = build_part("position", spec.position, env)
         tables = self.position.rotation_tables()
         if tables is None:
@@ -51,14 +62,19 @@ class GatedAttention(Mixer):
         self.cos, self.sin = tables
         if self.cos is not None and 2 * self.cos.shape[1] > spec.head_dim:
             raise ValueError(f"gated attention: {2 * self.cos.shape[1]} rotated dimensions do not fit a head of {spec.head_dim}")
-        self.w_in = self.w_o = self.q_norm = self.k_norm = self.sink = self.mix = None
+        self.w_in = self.w_o = self.q_norm = self.k_norm = self.sink = self.mix = self.bias = None
 
     @staticmethod
     def tensor_needs(spec: GatedAttentionSpec) -> List[TensorNeed]:
         H, G, dk, dv = spec.num_heads, spec.num_kv_heads, spec.head_dim, spec.value_dim
         out = [TensorNeed(spec.q_weight, (H * dk, spec.hidden)), TensorNeed(spec.o_weight, (spec.hidden, H * dv))]
         if spec.own_kv:
-            out += [TensorNeed(spec.k_weight, (G * dk, spec.hidden)), TensorNeed(spec.v_weight, (G * dv, spec.hidden))]
+            out.append(TensorNeed(spec.k_weight, (G * dk, spec.hidden)))
+            if not spec.keys_as_values:
+                out.append(TensorNeed(spec.v_weight, (G * dv, spec.hidden)))
+        for name, heads in ((spec.q_bias, H), (spec.k_bias if spec.own_kv else None, G)):
+            if name:
+                out.append(TensorNeed(name, (heads * dk,), "float32"))
         if spec.gate_weight:
             out.append(TensorNeed(spec.gate_weight, (H if spec.gate_per_head else H * dv, spec.hidden)))
         wide = spec.norm_scope == "projection"
@@ -90,7 +106,9 @@ class GatedAttention(Mixer):
 
     def load(self, tensors) -> None:
         s = self.spec
-        rows = [tensors[s.q_weight]] + ([tensors[s.k_weight], tensors[s.v_weight]] if s.own_kv else [])
+        rows = [tensors[s.q_weight]]
+        if s.own_kv:
+            rows += [tensors[s.k_weight]] + ([] if s.keys_as_values else [tensors[s.v_weight]])
         if s.gate_weight:
             rows.append(tensors[s.gate_weight])
         self.w_in = torch.cat(rows, dim=0).contiguous()  # one product for everything that reads the mixer's input
@@ -98,6 +116,11 @@ class GatedAttention(Mixer):
         self.q_norm = tensors[s.q_norm] if s.q_norm else None
         self.k_norm = tensors[s.k_norm] if s.k_norm else None
         self.sink = tensors[s.sink] if s.sink else None
+        if s.q_bias or (s.k_bias and s.own_kv):  # one vector over the columns [q | k], zeros where a projection has none
+            zeros = lambda heads: torch.zeros(heads * s.head_dim, dtype=torch.float32, device=self.env.device)  # noqa: E731
+            q_b = tensors[s.q_bias] if s.q_bias else zeros(s.num_heads)
+            k_b = [tensors[s.k_bias] if s.k_bias else zeros(s.num_kv_heads)] if s.own_kv else []
+            self.bias = torch.cat([q_b] + k_b).contiguous()
         self.mix = tensors[s.value_mix_weight].reshape(1) if s.value_mix == "mix" else None
         self.position.load(tensors)
 
@@ -126,10 +149,12 @@ class GatedAttention(Mixer):
         q = ctx.ws.get("gated_attention.q", (n, H * dk), dt)
         writes = cache.writes and cache.k is not None and s.own_kv
         wide = {"norm_wide": True} if s.norm_scope == "projection" else {}
+        if self.bias is not None or s.unit_rms or s.rot_pairs != "half" or s.keys_as_values:
+            wide = {"bias": self.bias, "unit_rms": s.unit_rms, "neighbours": s.rot_pairs == "neighbours", "keys_as_values": s.keys_as_values}
         ops.qkv_prep(parts, H, G if s.own_kv else 0, dk, dv, self.q_norm, self.k_norm, s.eps, self.cos, self.sin, ctx, ctx.block_tables[cache.group], q,
                      cache.k if writes else None, cache.v if writes else None, role, self.mix, v_first, **wide)
         att = ctx.ws.get("gated_attention.out", (n, H * dv), dt)
-        g_off = H * dk + (G * dk + G * dv if s.own_kv else 0)
+        g_off = H * dk + (G * dk + (0 if s.keys_as_values else G * dv) if s.own_kv else 0)
         ops.gated_attention(q, cache.k, cache.v, ctx, ctx.block_tables[cache.group], att, H, G, dk, dv, s.scale, s.window, s.chunk,
                             self.sink, parts if s.gate_weight else None, g_off, **({"gate_per_head": True} if s.gate_per_head else {}))
         return add_into_stream_or_partials(ops, att, self.w_o, ctx, False, "gated_attention.delta")

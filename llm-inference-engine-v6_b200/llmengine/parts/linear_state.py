@@ -1,5 +1,5 @@
 """Recurrent mixers whose memory is a matrix per head, S [dk, dv] in float32, kept in the request's state slot and updated token
-after token by a rank-one write k v^T (ops.linear_state). Four of them, which differ in what decays the matrix, what is
+after token by a rank-one write k v^T (ops.linear_state). Five of them, which differ in what decays the matrix, what is
 written, and what the projections read:
 
     Retention                q, k, v, g = W h;  q and k rotated at the token's position, k times a constant;  one decay a head
@@ -11,9 +11,11 @@ written, and what the projections read:
                              o = (S + diag(bonus) k v^T)^T r;  S <- diag(decay) S + k v^T
     GatedDelta               q, k, v behind a short causal convolution and silu (its last inputs kept in the slot), q and k unit
                              vectors per head; g, beta per head;  S <- g S;  w = beta (v - S^T k);  S <- S + k w^T;  o = S^T q
+    ChannelDelta             as GatedDelta with a decay per key channel, g = exp(-exp(A_log_h) softplus(W_a2 (W_a1 h) + dt_bias)):
+                             S <- diag(g) S;  w = beta (v - S^T k);  S <- S + k w^T;  o = S^T q
 
-All of them finish alike: every head's o divided by its root mean square, times a weight, times silu of a gate projection, then
-the output projection. Decays, gates, unit norms, the state and o are float32 in both engine precisions; the projections'
+All of them finish alike: every head's o divided by its root mean square, times a weight, times silu of a gate projection
+(ChannelDelta: sigmoid of a low-rank one), then the output projection. Decays, gates, unit norms, the state and o are float32 in both engine precisions; the projections'
 float32 sums are read as they come (K-split parts are added where they are read).
 """
 from __future__ import annotations
@@ -25,7 +27,7 @@ import torch
 from .attention import add_into_stream_or_partials, project_sums
 from .base import LayerCache, Mixer, NormalizedRows, StateNeed
 from .registry import build_part, part_class, register_part
-from .spec import DecayedLinearAttentionSpec, GatedDeltaSpec, RetentionSpec, TensorNeed, TokenShiftMixSpec
+from .spec import ChannelDeltaSpec, DecayedLinearAttentionSpec, GatedDeltaSpec, RetentionSpec, TensorNeed, TokenShiftMixSpec
 
 
 def _state_shape(env, heads: int, dk: int, dv: int):
@@ -234,7 +236,64 @@ class GatedDelta(Mixer):
         return add_into_stream_or_partials(ops, y, self.w_o, ctx, False, "delta.delta")
 
 
+class ChannelDelta(Mixer):
+    """The delta rule with a decay per head and key channel (ChannelDeltaSpec). One product for everything that reads the mixer's
+    input, [q | k | v | W_a1 h | W_g1 h | beta]; the short convolutions; both low-rank maps (decays, gate) in one launch; the state
+    under the rule "channel_delta", which takes beta's sums as they come; the heads' norm with a sigmoid gate."""
+
+    def __init__(self, spec: ChannelDeltaSpec, env):
+        super().__init__(spec, env)
+        if min(spec.heads, spec.kv_heads, spec.dim, spec.vdim, spec.taps, spec.decay_rank, spec.gate_rank) <= 0 or spec.heads % spec.kv_heads:
+            raise ValueError("channel delta rule: sizes must be positive and heads a multiple of kv_heads")
+        self.w_in = self.w_conv = self.w_a2_t = self.w_g2_t = self.a_log = self.dt_bias = self.norm_w = self.w_o = None
+
+    @staticmethod
+    def tensor_needs(spec: ChannelDeltaSpec) -> List[TensorNeed]:
+        H, G, dk, dv, D, K = spec.heads, spec.kv_heads, spec.dim, spec.vdim, spec.hidden, spec.taps
+        return [TensorNeed(spec.q_weight, (G * dk, D)), TensorNeed(spec.k_weight, (G * dk, D)), TensorNeed(spec.v_weight, (H * dv, D)),
+                TensorNeed(spec.q_conv, (G * dk, K), "float32"), TensorNeed(spec.k_conv, (G * dk, K), "float32"),
+                TensorNeed(spec.v_conv, (H * dv, K), "float32"), TensorNeed(spec.b_weight, (H, D)),
+                TensorNeed(spec.a1_weight, (spec.decay_rank, D)), TensorNeed(spec.a2_weight, (H * dk, spec.decay_rank)),
+                TensorNeed(spec.a_log, (H,), "float32"), TensorNeed(spec.dt_bias, (H * dk,), "float32"),
+                TensorNeed(spec.g1_weight, (spec.gate_rank, D)), TensorNeed(spec.g2_weight, (H * dv, spec.gate_rank)),
+                TensorNeed(spec.norm_weight, (dv,), "float32", init="around_one"), TensorNeed(spec.o_weight, (D, H * dv))]
+
+    def cache_needs(self):
+        s = self.spec
+        channels = 2 * s.kv_heads * s.dim + s.heads * s.vdim
+        return (StateNeed("channel_delta.state", _state_shape(self.env, s.heads, s.dim, s.vdim)),
+                StateNeed("channel_delta.conv", (s.taps - 1, channels)))
+
+    def load(self, tensors) -> None:
+        s = self.spec
+        self.w_in = torch.cat([tensors[n] for n in (s.q_weight, s.k_weight, s.v_weight, s.a1_weight, s.g1_weight, s.b_weight)], dim=0).contiguous()
+        self.w_conv = torch.cat([tensors[s.q_conv], tensors[s.k_conv], tensors[s.v_conv]], dim=0).contiguous()  # float32 [channels, taps]
+        self.w_a2_t, self.w_g2_t = tensors[s.a2_weight].t().contiguous(), tensors[s.g2_weight].t().contiguous()
+        self.a_log, self.dt_bias, self.norm_w, self.w_o = tensors[s.a_log], tensors[s.dt_bias], tensors[s.norm_weight], tensors[s.o_weight]
+
+    def forward(self, x, ctx, cache: LayerCache) -> Optional[torch.Tensor]:
+        s, ops, n, dt = self.spec, self.env.ops, ctx.n_tokens, self.env.dtype
+        if isinstance(x, NormalizedRows):
+            x = x.dense(ctx)
+        H, G, dk, dv = s.heads, s.kv_heads, s.dim, s.vdim
+        C = 2 * G * dk + H * dv
+        a_off, g_off, b_off = C, C + s.decay_rank, C + s.decay_rank + s.gate_rank
+        sums = project_sums(ops, ctx, x, self.w_in, "channel_delta.in")
+        qkv = ctx.ws.get("channel_delta.conv_out", (n, C), torch.float32)  # float32: what follows (unit norms, the recurrence) is
+        ops.conv_silu(sums, 0, C, self.w_conv, None, cache.states["channel_delta.conv"], ctx, qkv)
+        decay = ctx.ws.get("channel_delta.decay", (n, H * dk), torch.float32)
+        gate = ctx.ws.get("channel_delta.gate", (n, H * dv), torch.float32)
+        ops.channel_gates(sums, a_off, s.decay_rank, g_off, s.gate_rank, self.w_a2_t, self.w_g2_t, self.dt_bias, self.a_log, decay, gate, n)
+        o = ctx.ws.get("channel_delta.o", (n, H * dv), torch.float32)
+        ops.linear_state("channel_delta", qkv, 0, qkv, G * dk, qkv, 2 * G * dk, decay, 0, None, cache.states["channel_delta.state"], ctx, o,
+                         H, G, dk, dv, q_scale=dk ** -0.5, unit_eps=s.unit_eps, beta=sums, beta_off=b_off)
+        y = ctx.ws.get("channel_delta.y", (n, H * dv), dt)
+        ops.head_norm_gate(o, self.norm_w, gate, 0, s.eps, y, n, H, dv, act="sigmoid")
+        return add_into_stream_or_partials(ops, y, self.w_o, ctx, False, "channel_delta.delta")
+
+
 register_part("mixer", "retention", Retention)
 register_part("mixer", "decayed_linear_attention", DecayedLinearAttention)
 register_part("mixer", "token_shift_mix", TokenShiftMix)
 register_part("mixer", "gated_delta", GatedDelta)
+register_part("mixer", "channel_delta", ChannelDelta)

@@ -22,7 +22,11 @@ class RMSNorm(Norm):
         return [TensorNeed(spec.weight, (spec.dim,), "float32", init="around_one")]
 
     def load(self, tensors) -> None:
-        self.weight = tensors[self.spec.weight]
+        self.weight = self._gained(tensors[self.spec.weight])
+
+    def _gained(self, weight: torch.Tensor) -> torch.Tensor:
+        gain = float(self.spec.gain)
+        return weight if gain == 1.0 else (weight * gain).contiguous()
 
     can_defer = True
 
@@ -62,7 +66,7 @@ class UnitOffsetRMSNorm(RMSNorm):
         return [TensorNeed(spec.weight, (spec.dim,), "float32", init="normal")]
 
     def load(self, tensors) -> None:
-        self.weight = (tensors[self.spec.weight] + 1.0).contiguous()
+        self.weight = self._gained((tensors[self.spec.weight] + 1.0).contiguous())
 
 
 class LayerNorm(RMSNorm):

@@ -31,11 +31,14 @@ class TensorNeed:
 @dataclass(frozen=True)
 class NormSpec:
     """kind "rmsnorm": x / sqrt(mean(x^2) + eps) * weight. kind "rmsnorm_unit_offset": the same with the weight stored around
-    zero and applied as (1 + weight). kind "layernorm": (x - mean(x)) / sqrt(mean((x - mean(x))^2) + eps) * weight, no bias."""
+    zero and applied as (1 + weight). kind "layernorm": (x - mean(x)) / sqrt(mean((x - mean(x))^2) + eps) * weight, no bias.
+    gain: a constant of the model that multiplies what the norm hands on (a factor on the logits sits on the final norm: the head
+    is linear); it is folded into the weight when the weights are loaded."""
     kind: str
     dim: int
     eps: float
     weight: str  # checkpoint tensor name
+    gain: float = 1.0
 
 
 @dataclass(frozen=True)
@@ -78,7 +81,11 @@ class ScaledRotarySpec:
 class LatentAttentionSpec:
     """Causal attention whose keys and values are maps of one cached latent per token (parts/latent_attention.py).
     heads H; per head `dim` unrotated and `rot_dim` rotated query/key numbers and `vdim` value numbers;
-    `kv_rank` the latent of keys and values, `q_rank` the latent of queries. `scale` multiplies the scores as given."""
+    `kv_rank` the latent of keys and values, `q_rank` the latent of queries. `scale` multiplies the scores as given.
+    window: the last `window` tokens (0: all). sink: a number per head whose exponential is one more term of the softmax's
+    denominator. gate_per_head: the gate is one number a head (gate_weight [heads, hidden]) instead of one a result number.
+    own_kv False: the layer has no latent of its own (no dkv_weight, dkv_norm): its run reads the latents that the run named by
+    LayerRun.cache_from keeps. cache_window: as in GatedAttentionSpec."""
     kind: str
     hidden: int
     heads: int
@@ -93,13 +100,17 @@ class LatentAttentionSpec:
     dq_weight: str
     dq_norm: str
     uq_weight: str
-    dkv_weight: str
-    dkv_norm: str
+    dkv_weight: Optional[str]
+    dkv_norm: Optional[str]
     uk_weight: str
     uv_weight: str
     gate_weight: str
     o_weight: str
     window: int = 0
+    sink: Optional[str] = None
+    gate_per_head: bool = False
+    own_kv: bool = True
+    cache_window: Optional[int] = None
 
 
 @dataclass(frozen=True)
@@ -134,7 +145,11 @@ class GatedAttentionSpec:
     query heads' numbers together and one over all key heads', in place of a norm a head.
     own_kv False: the layer has no key and value projections (no k_weight, v_weight, k_norm): its run reads the cache of the run that
     LayerRun.cache_from names, keys as that layer normalised and rotated them. cache_window: how many of the last keys the cache
-    must keep when that is more than this layer's own window asks for, because borrowers look further back (None: `window`; 0: all)."""
+    must keep when that is more than this layer's own window asks for, because borrowers look further back (None: `window`; 0: all).
+    q_bias, k_bias: vectors added to the projections of queries and keys. rot_pairs: which numbers of a head turn together, "half"
+    (i with i + dims / 2) or "neighbours" (2i with 2i + 1). unit_rms: every query and key head is divided by its root mean square
+    over head_dim (eps inside the root, no weight) AFTER the rotation. keys_as_values: there is no value projection, a head's values
+    are its keys as the projection (with its bias) gives them, before any norm and rotation (value_dim == head_dim)."""
     kind: str
     hidden: int
     num_heads: int
@@ -146,7 +161,7 @@ class GatedAttentionSpec:
     position: object
     q_weight: str
     k_weight: str
-    v_weight: str
+    v_weight: Optional[str]
     o_weight: str
     q_norm: Optional[str] = None
     k_norm: Optional[str] = None
@@ -160,6 +175,11 @@ class GatedAttentionSpec:
     norm_scope: str = "head"               # "head" | "projection"
     own_kv: bool = True
     cache_window: Optional[int] = None
+    q_bias: Optional[str] = None
+    k_bias: Optional[str] = None
+    rot_pairs: str = "half"                # "half" | "neighbours"
+    unit_rms: bool = False
+    keys_as_values: bool = False
 
 
 @dataclass(frozen=True)
@@ -283,6 +303,41 @@ class GatedDeltaSpec:
     a_log: str
     dt_bias: str
     g_weight: str
+    norm_weight: str
+    o_weight: str
+    unit_eps: float = 1e-6
+
+
+@dataclass(frozen=True)
+class ChannelDeltaSpec:
+    """The delta rule with a decay per head and key channel behind short convolutions (kind "channel_delta", parts/linear_state.py):
+    q, k, v, beta, the convolutions and the unit norms as in GatedDeltaSpec; g = exp(-exp(a_log) * softplus(W_a2 (W_a1 h) +
+    dt_bias)) with a_log a number a head and dt_bias one a (head, key channel); S <- diag(g) S; w = beta (v - S^T k); S <- S + k w^T;
+    o = S^T q; every head's o is divided by its root mean square (eps) and multiplied by norm_weight [vdim];
+    out = Wo (o * sigmoid(W_g2 (W_g1 h))). decay_rank, gate_rank: rows of W_a1 and of W_g1."""
+    kind: str
+    hidden: int
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    taps: int
+    decay_rank: int
+    gate_rank: int
+    eps: float
+    q_weight: str
+    k_weight: str
+    v_weight: str
+    q_conv: str
+    k_conv: str
+    v_conv: str
+    b_weight: str
+    a1_weight: str
+    a2_weight: str
+    a_log: str
+    dt_bias: str
+    g1_weight: str
+    g2_weight: str
     norm_weight: str
     o_weight: str
     unit_eps: float = 1e-6
@@ -429,13 +484,20 @@ class LayerRun:
 @dataclass(frozen=True)
 class EmbeddingSpec:
     """kind "lookup": residual stream row = table row of the token id, widened to float32, times `scale`.
-    kind "lookup_normed": the same, then `norm` (any norm spec over `dim`) applied to the row: the stream starts normalised."""
+    kind "lookup_normed": the same, then `norm` (any norm spec over `dim`) applied to the row: the stream starts normalised.
+    kind "lookup_pairs": table row * scale + a row of a second table `pair_weight` [pair_buckets + 1, dim] that the token and the one
+    before it choose: (previous * pair_mul_prev + token * pair_mul_cur) mod pair_buckets, or row pair_buckets for a sequence's
+    first token. The previous token is kept in the request's slot."""
     weight: str
     vocab_size: int
     dim: int
     kind: str = "lookup"
     scale: float = 1.0
     norm: object = None
+    pair_weight: Optional[str] = None
+    pair_buckets: int = 0
+    pair_mul_prev: int = 0
+    pair_mul_cur: int = 0
 
 
 @dataclass(frozen=True)

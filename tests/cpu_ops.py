@@ -18,6 +18,19 @@ class CpuOps:
         out.copy_(table[ids[:n].long()].float() * scale)
         return out
 
+    def embed_pairs(self, table, pairs, buckets, mul_prev, mul_cur, scale, previous, batch, out):
+        for s in range(batch.n_seqs):
+            first, n, slot = int(batch.seq_qoff[s]), int(batch.seq_ntok[s]), int(batch.seq_slot[s])
+            before = int(previous[slot])
+            for t in range(first, first + n):
+                cur = int(batch.token_ids[t])
+                row = buckets if int(batch.positions[t]) == 0 else (before * mul_prev + cur * mul_cur) % buckets
+                out[t] = table[cur].float() * scale + pairs[row].float()
+                before = cur
+            if n > 0:
+                previous[slot] = before
+        return out
+
     def rmsnorm(self, h, weight, eps, out, delta=None, rows=None, n_rows=None, write_back=True, center=False):
         if rows is not None:
             n = rows.numel() if n_rows is None else n_rows
@@ -136,11 +149,11 @@ class CpuOps:
             assert page >= 0, "write into a page that was given back"
             cache[page, 0, pos % ps] = torch.cat([c[t], kr[t]]).to(cache.dtype)
 
-    def heads_product(self, a, w, out, gate=None, gate_off=0):
+    def heads_product(self, a, w, out, gate=None, gate_off=0, gate_per_head=False):
         y = torch.einsum("thk,hnk->thn", a.float(), w.float())
         if gate is not None:
             n, H, N = out.shape
-            g = gate.sum(0)[:n, gate_off:gate_off + H * N].view(n, H, N)
+            g = gate.sum(0)[:n, gate_off:gate_off + H].view(n, H, 1) if gate_per_head else gate.sum(0)[:n, gate_off:gate_off + H * N].view(n, H, N)
             y = y * torch.sigmoid(g)
         out.copy_(y.to(out.dtype))
         return out
@@ -161,7 +174,7 @@ class CpuOps:
         ql[:, :, kv_rank:] = r.to(ql.dtype)
         return ql
 
-    def latent_attention(self, ql, cache, batch, block_table, out, kv_rank, scale, window=0):
+    def latent_attention(self, ql, cache, batch, block_table, out, kv_rank, scale, window=0, sink=None):
         ps = cache.shape[2]
         for t in range(batch.n_tokens):
             pos = int(batch.positions[t])
@@ -170,7 +183,8 @@ class CpuOps:
             pages = block_table[int(batch.token_seq[t])][(idx // ps).long()].long()
             assert (pages >= 0).all(), "read from a page that was given back"
             rows = cache[pages, 0, (idx % ps).long(), :].float()  # [S, Dk]
-            p = torch.softmax((ql[t].float() @ rows.t()) * scale, dim=-1)  # [H, S]
+            s = (ql[t].float() @ rows.t()) * scale  # [H, S]
+            p = torch.softmax(s if sink is None else torch.cat([s, sink[:, None]], dim=1), dim=-1)[:, :s.shape[1]]
             out[t] = (p @ rows[:, :kv_rank]).to(out.dtype)
         return out
 
@@ -298,24 +312,32 @@ class CpuOps:
         return h
 
     def qkv_prep(self, parts, heads, kv_heads, dk, dv, q_norm, k_norm, eps, cos, sin, batch, block_table, q_out, kcache, vcache,
-                 mix_role=0, mix_weight=None, v_first=None, norm_wide=False):
+                 mix_role=0, mix_weight=None, v_first=None, norm_wide=False, bias=None, neighbours=False, unit_rms=False,
+                 keys_as_values=False):
         src = parts.sum(0)
+        if bias is not None:
+            src = src.clone()
+            src[:, :bias.numel()] += bias
         half = 0 if cos is None else cos.shape[1]
         for t in range(batch.n_tokens):
             pos = int(batch.positions[t])
             row = src[t].float()
             q = row[:heads * dk].view(heads, dk).clone()
             k = row[heads * dk:(heads + kv_heads) * dk].view(kv_heads, dk).clone()
-            v = row[(heads + kv_heads) * dk:(heads + kv_heads) * dk + kv_heads * dv].clone()
+            v = k.reshape(-1).clone() if keys_as_values else row[(heads + kv_heads) * dk:(heads + kv_heads) * dk + kv_heads * dv].clone()
             for x, w in ((q, q_norm), (k, k_norm)):
                 if w is not None and x.numel() and norm_wide:  # one norm over the whole projection, a weight a number
                     x.copy_(x / torch.sqrt((x * x).mean() + eps) * w.view(x.shape))
                 elif w is not None and x.numel():
                     x.copy_(x / torch.sqrt((x * x).mean(-1, keepdim=True) + eps) * w)
                 if half:
-                    a, b = x[:, :half].clone(), x[:, half:2 * half].clone()
-                    x[:, :half] = a * cos[pos] - b * sin[pos]
-                    x[:, half:2 * half] = b * cos[pos] + a * sin[pos]
+                    ia = slice(0, 2 * half, 2) if neighbours else slice(0, half)
+                    ib = slice(1, 2 * half, 2) if neighbours else slice(half, 2 * half)
+                    a, b = x[:, ia].clone(), x[:, ib].clone()
+                    x[:, ia] = a * cos[pos] - b * sin[pos]
+                    x[:, ib] = b * cos[pos] + a * sin[pos]
+                if unit_rms and x.numel():
+                    x.copy_(x / torch.sqrt((x * x).mean(-1, keepdim=True) + eps))
             if mix_role == 1:
                 v_first[t] = v
             elif mix_role == 2:
@@ -425,11 +447,12 @@ class CpuOps:
         return (t if t.dim() == 2 else t.sum(0))[:, off:off + width]
 
     def linear_state(self, rule, q, q_off, k, k_off, v, v_off, decay, decay_off, bonus, state, batch, out, heads, kv_heads, dk, dv,
-                     q_scale=1.0, unit_eps=-1.0, decay_const=False):
+                     q_scale=1.0, unit_eps=-1.0, decay_const=False, beta=None, beta_off=0):
         Q = self._cols(q, q_off, kv_heads * dk).reshape(-1, kv_heads, dk) * q_scale
         K = self._cols(k, k_off, kv_heads * dk).reshape(-1, kv_heads, dk)
         V = self._cols(v, v_off, heads * dv).reshape(-1, heads, dv)
-        if rule == "delta" and unit_eps >= 0:
+        strength = torch.sigmoid(self._cols(beta, beta_off, heads)) if beta is not None else None
+        if rule in ("delta", "channel_delta") and unit_eps >= 0:
             Q = Q / torch.sqrt((Q / q_scale).pow(2).sum(-1, keepdim=True) + unit_eps)
             K = K / torch.sqrt(K.pow(2).sum(-1, keepdim=True) + unit_eps)
         rep = heads // kv_heads
@@ -443,6 +466,11 @@ class CpuOps:
                     g, beta = decay[t, decay_off:decay_off + heads], decay[t, decay_off + heads:decay_off + 2 * heads]
                     S = S * g[:, None, None]
                     w = beta[:, None] * (vt - torch.einsum("hkv,hk->hv", S, kt))
+                    S = S + kt[:, :, None] * w[:, None, :]
+                    o = torch.einsum("hkv,hk->hv", S, qt)
+                elif rule == "channel_delta":
+                    S = S * decay[t, decay_off:decay_off + heads * dk].view(heads, dk)[:, :, None]
+                    w = strength[t][:, None] * (vt - torch.einsum("hkv,hk->hv", S, kt))
                     S = S + kt[:, :, None] * w[:, None, :]
                     o = torch.einsum("hkv,hk->hv", S, qt)
                 else:
@@ -488,12 +516,19 @@ class CpuOps:
         out[:n_tokens, H:] = torch.sigmoid(self._cols(b, b_off, H)[:n_tokens])
         return out
 
-    def head_norm_gate(self, o, weight, gate, gate_off, eps, out, n_tokens, heads, dv):
+    def channel_gates(self, sums, decay_col, decay_rank, gate_col, gate_rank, decay_t, gate_t, dt_bias, a_log, decay, gate, n_tokens):
+        z = self._cols(sums, decay_col, decay_rank)[:n_tokens] @ decay_t.float() + dt_bias
+        rate = torch.exp(a_log).repeat_interleave(decay_t.shape[1] // a_log.numel())
+        decay[:n_tokens] = torch.exp(-rate * torch.nn.functional.softplus(z))
+        gate[:n_tokens] = self._cols(sums, gate_col, gate_rank)[:n_tokens] @ gate_t.float()
+
+    def head_norm_gate(self, o, weight, gate, gate_off, eps, out, n_tokens, heads, dv, act="silu"):
         y = o[:n_tokens].view(n_tokens, heads, dv)
         y = y / torch.sqrt((y * y).mean(-1, keepdim=True) + eps) * (weight.view(heads, dv) if weight.numel() == heads * dv and heads > 1 else weight)
         y = y.reshape(n_tokens, heads * dv)
         if gate is not None:
-            y = y * torch.nn.functional.silu(self._cols(gate, gate_off, heads * dv)[:n_tokens])
+            g = self._cols(gate, gate_off, heads * dv)[:n_tokens]
+            y = y * (torch.sigmoid(g) if act == "sigmoid" else torch.nn.functional.silu(g))
         out[:n_tokens] = y.to(out.dtype)
         return out
 
