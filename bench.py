@@ -532,7 +532,34 @@ SOGUTAR_SIZES = {
     "w1024": (sogutar_sizes(1024, 16, 4, 64, 1024, 8, 128, 2816, 8, 2, 2, 1408, 1408, 4, 32768), SELINEX_SIZES["w1024"][0]),
     "w2048": (sogutar_sizes(2048, 32, 8, 64, 1024, 16, 128, 8192, 16, 2, 4, 2048, 2048, 4, 32768), SELINEX_SIZES["w2048"][0]),
 }
-DESIGNS = {"vapelix": DESIGN_SIZES, "zulopel": ZULOPEL_SIZES, "selinex": SELINEX_SIZES, "sogutar": SOGUTAR_SIZES}
+
+
+def zudatar_sizes(width, heads, kv_heads, dim, window, lat_heads, lat_dim, kv_rank, q_rank, state_heads, state_dim, rank, ff, layers, vocab):
+    att = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "mask": {"size": window},
+           "rot": {"dims": dim // 2, "base": 500000.0}}
+    lat = {"heads": lat_heads, "dim": lat_dim, "vdim": lat_dim, "kv_rank": kv_rank, "q_rank": q_rank, "scale": lat_dim ** -0.5, "mask": {"size": window}}
+    delta = {"heads": state_heads, "kv_heads": state_heads, "dim": state_dim, "vdim": state_dim, "conv": 4, "decay_rank": rank, "gate_rank": rank}
+    dense = {"kind": "dense", "ff": ff}
+    kinds = [("channel_delta", delta), ("attention", att), ("latent_attention", lat), ("latent_attention", dict(lat, kv_from=2))]
+    return {"architecture": "Zudatar", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "logit_scale": 0.25, "max_positions": 8192,
+            "embedding": {"scale": width ** 0.5, "bigram": {"buckets": vocab - 1, "mul_prev": 1009, "mul_cur": 31}},
+            "layers": [{"type": t, "mixer": m, "mlp": dense} for t, m in (kinds[i % 4] for i in range(layers))]}
+
+
+def sogutar_dense(cfg):
+    """The Sogutar configuration with a dense feed-forward of one size in every layer."""
+    dense = next(l["mlp"] for l in cfg["layers"] if l["mlp"]["kind"] == "dense")
+    return dict(cfg, layers=[dict(l, mlp=dense) for l in cfg["layers"]])
+
+
+# Zudatar: a delta-rule layer with a decay a channel, windowed attention whose values are its keys, and two latent-attention layers of
+# which the second reads the first one's latents, dense feed-forwards; beside it the Sogutar configuration of the same name with
+# dense feed-forwards (one mixer a layer, windowed attention, borrowed keys, a matrix of state a head: the closest existing model)
+ZUDATAR_SIZES = {
+    "w1024": (zudatar_sizes(1024, 16, 4, 64, 1024, 8, 64, 256, 384, 8, 128, 64, 2816, 4, 32768), sogutar_dense(SOGUTAR_SIZES["w1024"][0])),
+    "w2048": (zudatar_sizes(2048, 32, 8, 64, 1024, 16, 128, 512, 768, 16, 128, 128, 8192, 4, 32768), sogutar_dense(SOGUTAR_SIZES["w2048"][0])),
+}
+DESIGNS = {"vapelix": DESIGN_SIZES, "zulopel": ZULOPEL_SIZES, "selinex": SELINEX_SIZES, "sogutar": SOGUTAR_SIZES, "zudatar": ZUDATAR_SIZES}
 
 
 def run_design(args):

@@ -33,6 +33,7 @@ constexpr int LS_THREADS = 128;   // threads that hold the state, at most: fewer
 constexpr int LS_FETCHERS = 128;  // threads behind them that fetch the tiles of tokens ahead
 constexpr int LS_BLOCK = LS_THREADS + LS_FETCHERS;
 constexpr int LS_BUFFERS = 3;    // tiles in shared memory: walked, landing, issued
+constexpr size_t LS_SMEM = 112 * 1024;  // of the tiles, at most (portions)
 
 __device__ __forceinline__ float parts_sum(const float* __restrict__ p, int n_parts, size_t pstride, size_t i) {
   float s = p[i];
@@ -510,6 +511,84 @@ __global__ void __launch_bounds__(128) channel_gates_kernel(const ChannelGates p
   }
 }
 
+// The same maps for prompt-sized steps in bfloat16, on tensor cores: a block takes 64 tokens x 128 channels of one map, eight warps
+// of 16 x 64 each; w0 [C0, R0], w1 [C1, R1] as the checkpoint stores them. The low-rank numbers enter as the sum of two bfloat16
+// numbers (the number rounded, and what the rounding left), a product each, so they count with about 16 bits of mantissa.
+constexpr int CG_TOK = 64, CG_COLS = 128, CG_K = 64, CG_LD = CG_K + 8, CG_THREADS = 256;
+__global__ void __launch_bounds__(CG_THREADS) channel_gates_mma_kernel(const ChannelGates p, const bf16* __restrict__ w0, const bf16* __restrict__ w1) {
+  __shared__ __align__(16) bf16 hi_s[CG_TOK][CG_LD], lo_s[CG_TOK][CG_LD], w_s[CG_COLS][CG_LD];
+  dep_launch();
+  dep_wait();
+  const int blocks0 = (p.C0 + CG_COLS - 1) / CG_COLS;
+  const bool first = (int)blockIdx.x < blocks0;
+  const Sums x = first ? p.x0 : p.x1;
+  const bf16* w = first ? w0 : w1;
+  const int R = first ? p.R0 : p.R1, C = first ? p.C0 : p.C1, c0 = ((int)blockIdx.x - (first ? 0 : blocks0)) * CG_COLS;
+  const int t0 = blockIdx.y * CG_TOK, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, wm = warp & 3, wn = warp >> 2;
+  float acc[8][4];
+#pragma unroll
+  for (int j = 0; j < 8; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f;
+  const bool quads = R % 8 == 0 && (reinterpret_cast<uintptr_t>(w) & 15u) == 0;
+  for (int k0 = 0; k0 < R; k0 += CG_K) {
+    if (k0 > 0) __syncthreads();  // everyone is done with the block before
+    for (int i = tid; i < CG_TOK * CG_K; i += CG_THREADS) {
+      const int t = i / CG_K, k = i % CG_K;
+      float v = 0.f;
+      if (t0 + t < p.n_tokens && k0 + k < R) v = parts_sum(x.p, x.n, x.stride, (size_t)(t0 + t) * x.width + x.off + k0 + k);
+      const bf16 h = __float2bfloat16_rn(v);
+      hi_s[t][k] = h;
+      lo_s[t][k] = __float2bfloat16_rn(v - __bfloat162float(h));
+    }
+    if (quads) {
+      for (int i = tid; i < CG_COLS * (CG_K / 8); i += CG_THREADS) {
+        const int c = i / (CG_K / 8), k = (i % (CG_K / 8)) * 8;
+        uint4 v = make_uint4(0, 0, 0, 0);
+        if (c0 + c < C && k0 + k < R) v = *reinterpret_cast<const uint4*>(w + (size_t)(c0 + c) * R + k0 + k);
+        *reinterpret_cast<uint4*>(&w_s[c][k]) = v;
+      }
+    } else {
+      for (int i = tid; i < CG_COLS * CG_K; i += CG_THREADS) {
+        const int c = i / CG_K, k = i % CG_K;
+        w_s[c][k] = (c0 + c < C && k0 + k < R) ? w[(size_t)(c0 + c) * R + k0 + k] : __float2bfloat16_rn(0.f);
+      }
+    }
+    __syncthreads();
+#pragma unroll
+    for (int ks = 0; ks < CG_K / 16; ++ks) {
+      if (k0 + ks * 16 >= R) break;
+      uint32_t ah[4], al[4];
+      ldmatrix_x4(ah, &hi_s[wm * 16 + (lane % 16)][ks * 16 + (lane / 16) * 8]);
+      ldmatrix_x4(al, &lo_s[wm * 16 + (lane % 16)][ks * 16 + (lane / 16) * 8]);
+#pragma unroll
+      for (int j2 = 0; j2 < 4; ++j2) {
+        uint32_t b[4];
+        ldmatrix_x4(b, &w_s[wn * 64 + j2 * 16 + (lane % 8) + (lane / 16) * 8][ks * 16 + ((lane / 8) % 2) * 8]);
+        mma_bf16(acc[2 * j2], al, b[0], b[1]);
+        mma_bf16(acc[2 * j2], ah, b[0], b[1]);
+        mma_bf16(acc[2 * j2 + 1], al, b[2], b[3]);
+        mma_bf16(acc[2 * j2 + 1], ah, b[2], b[3]);
+      }
+    }
+  }
+#pragma unroll
+  for (int j = 0; j < 8; ++j) {
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      const int c = c0 + wn * 64 + j * 8 + 2 * (lane % 4) + e;
+      if (c >= C) continue;
+      const float b = first ? p.bias0[c] : 0.f, rate = first ? expf(p.a_log[c / p.per]) : 0.f;
+#pragma unroll
+      for (int half = 0; half < 2; ++half) {
+        const int t = t0 + wm * 16 + lane / 4 + half * 8;
+        if (t >= p.n_tokens) continue;
+        const float z = acc[j][2 * half + e] + b;
+        if (first) p.out0[(size_t)t * C + c] = expf(-rate * (z > 20.0f ? z : log1pf(expf(z))));
+        else p.out1[(size_t)t * C + c] = z;
+      }
+    }
+  }
+}
+
 // a warp a (token, head): out = o / sqrt(mean(o^2) + eps) * weight * act(gate), act silu or sigmoid; weight [dv] for all heads or
 // [H * dv]
 template <typename T>
@@ -615,8 +694,10 @@ extern "C" int llm_linear_state(int mode, const float* q, int qn, long long qs, 
   };
   const bool few = n_tokens <= 2 * n_seqs;
   p.tile = few ? 2 : 16;
-  while (p.tile > 1 && smem_for(p.tile) > 48 * 1024) p.tile /= 2;
-  LLM_REQUIRE(smem_for(p.tile) <= 48 * 1024, "linear_state: heads of %d / %d numbers exceed one block's shared memory", dk, dv);
+  // a portion's blocks have a multiprocessor each, so they may take more than the default 48 KB: longer tiles, fewer meetings
+  const size_t smem_limit = few ? 48 * 1024 : LS_SMEM;
+  while (p.tile > 1 && smem_for(p.tile) > smem_limit) p.tile /= 2;
+  LLM_REQUIRE(smem_for(p.tile) <= smem_limit, "linear_state: heads of %d / %d numbers exceed one block's shared memory", dk, dv);
   p.one_part = qn == 1 && kn == 1 && vn == 1 && (mode != 3 || bn == 1);
   auto quads = [](const void* ptr, long long width, long long off) { return ((uintptr_t)ptr & 15) == 0 && width % 4 == 0 && off % 4 == 0; };
   p.vec4 = dk % 4 == 0 && dv % 4 == 0 && quads(q, qw, qo) && quads(k, kw, ko) && quads(v, vw, vo) && (mode == 2 || quads(decay, p.decay_width, decay_off));
@@ -626,9 +707,14 @@ extern "C" int llm_linear_state(int mode, const float* q, int qn, long long qs, 
   while (p.walkers > 32 && 2 * per_column_block * ceil_div(dv, p.walkers / p.R) <= device_sms()) p.walkers /= 2;
   dim3 grid(ceil_div(dv, p.walkers / p.R), H, n_seqs);
   const size_t smem = smem_for(p.tile);
-#define LS_LAUNCH(M, RR)                                                                                        \
-  if (few) launch_kernel(linear_state_kernel<M, RR, true>, grid, p.walkers + LS_FETCHERS, smem, stream, p);     \
-  else launch_kernel(linear_state_kernel<M, RR, false>, grid, p.walkers + LS_FETCHERS, smem, stream, p)
+#define LS_LAUNCH(M, RR)                                                                                                              \
+  if (few) {                                                                                                                         \
+    launch_kernel(linear_state_kernel<M, RR, true>, grid, p.walkers + LS_FETCHERS, smem, stream, p);                                 \
+  } else {                                                                                                                           \
+    LLM_REQUIRE(smem <= 48 * 1024 || cudaFuncSetAttribute(linear_state_kernel<M, RR, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, \
+                                                          (int)LS_SMEM) == cudaSuccess, "linear_state: cannot raise the shared memory limit"); \
+    launch_kernel(linear_state_kernel<M, RR, false>, grid, p.walkers + LS_FETCHERS, smem, stream, p);                                \
+  }
 #define LS_LANES(M)                  \
   switch (p.R) {                     \
     case 1: LS_LAUNCH(M, 1); break;  \
@@ -677,9 +763,10 @@ extern "C" int llm_delta_gates(const float* a, int an, long long as, int aw, int
   return LLM_OK;
 }
 
-// x: float32 sums; columns x0.. (R0 of them) and x1.. (R1). wt0 [R0, C0], wt1 [R1, C1]: the maps transposed, in the engine's dtype.
+// x: float32 sums; columns x0.. (R0 of them) and x1.. (R1). wt0 [R0, C0], wt1 [R1, C1]: the maps transposed, in the engine's dtype;
+// w0, w1 (bfloat16 alone, or null): the maps as they are stored, for steps of more than 64 tokens on tensor cores.
 extern "C" int llm_channel_gates(const float* x, int xn, long long xs, int xw, int x0, int x1, int R0, int R1, const void* wt0, const void* wt1,
-                                 const float* bias0, const float* a_log, int C0, int C1, int per, float* out0, float* out1, int dtype,
+                                 const void* w0, const void* w1, const float* bias0, const float* a_log, int C0, int C1, int per, float* out0, float* out1, int dtype,
                                  int n_tokens, cudaStream_t stream) {
   if (n_tokens == 0) return LLM_OK;
   LLM_REQUIRE(n_tokens > 0 && x && xn >= 1 && wt0 && wt1 && bias0 && a_log && out0 && out1, "channel_gates: missing tensors");
@@ -689,6 +776,13 @@ extern "C" int llm_channel_gates(const float* x, int xn, long long xs, int xw, i
   ChannelGates p;
   p.x0 = Sums{x, xn, (size_t)xs, xw, x0}; p.x1 = Sums{x, xn, (size_t)xs, xw, x1};
   p.R0 = R0; p.R1 = R1; p.C0 = C0; p.C1 = C1; p.per = per; p.bias0 = bias0; p.a_log = a_log; p.out0 = out0; p.out1 = out1; p.n_tokens = n_tokens;
+  if (dtype == LLM_BF16 && w0 && w1 && n_tokens > 64) {
+    dim3 tiles(ceil_div(C0, CG_COLS) + ceil_div(C1, CG_COLS), ceil_div(n_tokens, CG_TOK));
+    LLM_REQUIRE(tiles.y <= 65535, "channel_gates: too many tokens in one step (%d)", n_tokens);
+    launch_kernel(channel_gates_mma_kernel, tiles, CG_THREADS, 0, stream, p, (const bf16*)w0, (const bf16*)w1);
+    LLM_CHECK_LAUNCH("channel_gates");
+    return LLM_OK;
+  }
   const size_t smem = ((size_t)max(R0, R1) * 8 + 4 * 32 * 8) * sizeof(float);
   LLM_REQUIRE(smem <= 48 * 1024, "channel_gates: ranks of %d / %d exceed one block's shared memory", R0, R1);
   dim3 grid(ceil_div(C0, 32) + ceil_div(C1, 32), ceil_div(n_tokens, 8));

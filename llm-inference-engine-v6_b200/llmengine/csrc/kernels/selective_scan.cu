@@ -69,6 +69,46 @@ __global__ void conv_silu_kernel(const float* __restrict__ parts, int n_parts, s
   }
 }
 
+// The same for prompt-sized steps whose product comes in one part: a thread walks RUN tokens of a channel with the taps' inputs and
+// weights in registers, so every input is read once (and the first taps - 1 of a run once more). The additions of a token are those
+// of the kernel above, in the same order.
+template <typename T, int K, int RUN>
+__global__ void __launch_bounds__(256)
+    conv_silu_run_kernel(const float* __restrict__ x, int width, int x_off, int C, const T* __restrict__ w, const float* __restrict__ bias,
+                         const float* __restrict__ conv_state, const int* __restrict__ token_seq, const int* __restrict__ seq_qoff,
+                         const int* __restrict__ seq_slot, T* __restrict__ out, int n_tokens) {
+  dep_launch();
+  dep_wait();
+  const int c = blockIdx.x * blockDim.x + threadIdx.x;
+  if (c >= C) return;
+  const int t0 = blockIdx.y * RUN, t1 = min(n_tokens, t0 + RUN);
+  float wt[K], in[K];  // in[j]: the input that tap j meets
+#pragma unroll
+  for (int j = 0; j < K; ++j) wt[j] = to_f32(w[(size_t)c * K + j]);
+  const float b = bias ? bias[c] : 0.f;
+  int seq = -1;
+#pragma unroll 4
+  for (int tok = t0; tok < t1; ++tok) {
+    if (token_seq[tok] != seq) {  // the run's first token, or a request's: what lies before it comes from the step or the slot
+      seq = token_seq[tok];
+      const int first = seq_qoff[seq];
+      const float* st = conv_state + (size_t)seq_slot[seq] * (K - 1) * C;
+#pragma unroll
+      for (int j = 0; j < K - 1; ++j) {
+        const int src = tok - (K - 1) + j;
+        in[j + 1] = src >= first ? x[(size_t)src * width + x_off + c] : st[(size_t)((K - 1) + (src - first)) * C + c];
+      }
+    }
+#pragma unroll
+    for (int j = 0; j < K - 1; ++j) in[j] = in[j + 1];
+    in[K - 1] = x[(size_t)tok * width + x_off + c];
+    float acc = b;
+#pragma unroll
+    for (int j = 0; j < K; ++j) acc = fmaf(wt[j], in[j], acc);
+    out[(size_t)tok * C + c] = from_f32<T>(silu_f(acc));
+  }
+}
+
 __global__ void conv_state_kernel(const float* __restrict__ parts, int n_parts, size_t pstride, int width, int x_off, int C, int K,
                                   float* __restrict__ conv_state, const int* __restrict__ seq_qoff, const int* __restrict__ seq_ntok,
                                   const int* __restrict__ seq_slot, int n_seqs) {
@@ -370,7 +410,18 @@ extern "C" int llm_conv_silu(const float* parts, int n_parts, long long pstride,
   LLM_REQUIRE(n_tokens > 0 && n_seqs > 0 && n_parts >= 1 && C > 0 && K >= 1 && K <= MAX_TAPS, "conv_silu: bad sizes (taps %d, at most %d)", K, MAX_TAPS);
   LLM_REQUIRE(x_off >= 0 && x_off + C <= width, "conv_silu: columns outside the product");
   dim3 grid(ceil_div(C, 256), n_tokens < 65535 ? n_tokens : 65535);
-  if (dtype == LLM_F32)
+  constexpr int RUN = 16;
+  const bool runs = n_parts == 1 && n_tokens > 64 && K >= 2 && K <= 4 && ceil_div(n_tokens, RUN) <= 65535;
+  if (runs && (dtype == LLM_F32 || dtype == LLM_BF16)) {
+    dim3 run_grid(ceil_div(C, 256), ceil_div(n_tokens, RUN));
+#define LLM_CONV_RUN(T, KK)                                                                                                             \
+  launch_kernel(conv_silu_run_kernel<T, KK, RUN>, run_grid, 256, 0, stream, parts, width, x_off, C, (const T*)w, bias, (const float*)conv_state, \
+                token_seq, seq_qoff, seq_slot, (T*)out, n_tokens)
+#define LLM_CONV_TAPS(T) if (K == 2) LLM_CONV_RUN(T, 2); else if (K == 3) LLM_CONV_RUN(T, 3); else LLM_CONV_RUN(T, 4)
+    if (dtype == LLM_F32) { LLM_CONV_TAPS(float); } else { LLM_CONV_TAPS(bf16); }
+#undef LLM_CONV_TAPS
+#undef LLM_CONV_RUN
+  } else if (dtype == LLM_F32)
     launch_kernel(conv_silu_kernel<float>, grid, 256, 0, stream, parts, n_parts, (size_t)pstride, width, x_off, C, K,
                   (const float*)w, bias, (const float*)conv_state, token_seq, seq_qoff, seq_slot, (float*)out, n_tokens);
   else if (dtype == LLM_BF16)

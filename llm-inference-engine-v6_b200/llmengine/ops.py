@@ -1455,11 +1455,13 @@ class CudaOps:
         return out
 
     def channel_gates(self, sums, decay_col: int, decay_rank: int, gate_col: int, gate_rank: int, decay_t: torch.Tensor, gate_t: torch.Tensor,
-                      dt_bias: torch.Tensor, a_log: torch.Tensor, decay: torch.Tensor, gate: torch.Tensor, n_tokens: int) -> None:
+                      dt_bias: torch.Tensor, a_log: torch.Tensor, decay: torch.Tensor, gate: torch.Tensor, n_tokens: int,
+                      decay_w: Optional[torch.Tensor] = None, gate_w: Optional[torch.Tensor] = None) -> None:
         """Two low-rank maps of the float32 `sums` [parts, n, width] in one launch: decay[t, c] = exp(-exp(a_log[c // per]) *
         softplus(dt_bias[c] + sum_r decay_t[r, c] * sums[t, decay_col + r])) with per = channels / len(a_log), and
         gate[t, c] = sum_r gate_t[r, c] * sums[t, gate_col + r]. decay_t, gate_t [rank, channels]: the maps stored transposed;
-        decay, gate: float32 [n, channels]."""
+        decay, gate: float32 [n, channels]. decay_w, gate_w [channels, rank] (optional): the maps as they are stored; with them a
+        bfloat16 step of more than 64 tokens runs on tensor cores."""
         for t, name in ((dt_bias, "dt_bias"), (a_log, "a_log"), (decay, "decay"), (gate, "gate")):
             _need(t, "channel_gates." + name, torch.float32)
             assert t.is_contiguous()
@@ -1468,10 +1470,14 @@ class CudaOps:
         assert decay_t.is_contiguous() and gate_t.is_contiguous() and decay_t.shape[0] == decay_rank and gate_t.shape[0] == gate_rank
         assert dt_bias.numel() == C0 and C0 % a_log.numel() == 0 and decay.shape[1] == C0 and gate.shape[1] == C1
         assert decay.shape[0] >= n_tokens and gate.shape[0] >= n_tokens
+        mma = self.tensor_cores and decay_w is not None and gate_w is not None and decay_w.dtype == torch.bfloat16
+        if mma:
+            assert decay_w.is_contiguous() and gate_w.is_contiguous() and decay_w.shape == (C0, decay_rank) and gate_w.shape == (C1, gate_rank)
         p, parts, stride, width, _ = self._sums(sums, 0, "channel_gates.sums")
         lib = self.lib()
         self._check(lib.llm_channel_gates(p, parts, stride, width, c_int(decay_col), c_int(gate_col), c_int(decay_rank), c_int(gate_rank),
-                                          _ptr(decay_t), _ptr(gate_t), _ptr(dt_bias), _ptr(a_log), c_int(C0), c_int(C1),
+                                          _ptr(decay_t), _ptr(gate_t), _ptr(decay_w if mma else None), _ptr(gate_w if mma else None),
+                                          _ptr(dt_bias), _ptr(a_log), c_int(C0), c_int(C1),
                                           c_int(C0 // a_log.numel()), _ptr(decay), _ptr(gate), c_int(dtype_code(decay_t.dtype)), c_int(n_tokens),
                                           _stream()), lib)
 

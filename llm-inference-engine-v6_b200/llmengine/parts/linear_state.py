@@ -245,7 +245,7 @@ class ChannelDelta(Mixer):
         super().__init__(spec, env)
         if min(spec.heads, spec.kv_heads, spec.dim, spec.vdim, spec.taps, spec.decay_rank, spec.gate_rank) <= 0 or spec.heads % spec.kv_heads:
             raise ValueError("channel delta rule: sizes must be positive and heads a multiple of kv_heads")
-        self.w_in = self.w_conv = self.w_a2_t = self.w_g2_t = self.a_log = self.dt_bias = self.norm_w = self.w_o = None
+        self.w_in = self.w_conv = self.w_a2 = self.w_g2 = self.w_a2_t = self.w_g2_t = self.a_log = self.dt_bias = self.norm_w = self.w_o = None
 
     @staticmethod
     def tensor_needs(spec: ChannelDeltaSpec) -> List[TensorNeed]:
@@ -268,7 +268,8 @@ class ChannelDelta(Mixer):
         s = self.spec
         self.w_in = torch.cat([tensors[n] for n in (s.q_weight, s.k_weight, s.v_weight, s.a1_weight, s.g1_weight, s.b_weight)], dim=0).contiguous()
         self.w_conv = torch.cat([tensors[s.q_conv], tensors[s.k_conv], tensors[s.v_conv]], dim=0).contiguous()  # float32 [channels, taps]
-        self.w_a2_t, self.w_g2_t = tensors[s.a2_weight].t().contiguous(), tensors[s.g2_weight].t().contiguous()
+        self.w_a2, self.w_g2 = tensors[s.a2_weight], tensors[s.g2_weight]
+        self.w_a2_t, self.w_g2_t = self.w_a2.t().contiguous(), self.w_g2.t().contiguous()
         self.a_log, self.dt_bias, self.norm_w, self.w_o = tensors[s.a_log], tensors[s.dt_bias], tensors[s.norm_weight], tensors[s.o_weight]
 
     def forward(self, x, ctx, cache: LayerCache) -> Optional[torch.Tensor]:
@@ -283,7 +284,8 @@ class ChannelDelta(Mixer):
         ops.conv_silu(sums, 0, C, self.w_conv, None, cache.states["channel_delta.conv"], ctx, qkv)
         decay = ctx.ws.get("channel_delta.decay", (n, H * dk), torch.float32)
         gate = ctx.ws.get("channel_delta.gate", (n, H * dv), torch.float32)
-        ops.channel_gates(sums, a_off, s.decay_rank, g_off, s.gate_rank, self.w_a2_t, self.w_g2_t, self.dt_bias, self.a_log, decay, gate, n)
+        ops.channel_gates(sums, a_off, s.decay_rank, g_off, s.gate_rank, self.w_a2_t, self.w_g2_t, self.dt_bias, self.a_log, decay, gate, n,
+                          decay_w=self.w_a2, gate_w=self.w_g2)
         o = ctx.ws.get("channel_delta.o", (n, H * dv), torch.float32)
         ops.linear_state("channel_delta", qkv, 0, qkv, G * dk, qkv, 2 * G * dk, decay, 0, None, cache.states["channel_delta.state"], ctx, o,
                          H, G, dk, dv, q_scale=dk ** -0.5, unit_eps=s.unit_eps, beta=sums, beta_off=b_off)

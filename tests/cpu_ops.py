@@ -516,7 +516,8 @@ class CpuOps:
         out[:n_tokens, H:] = torch.sigmoid(self._cols(b, b_off, H)[:n_tokens])
         return out
 
-    def channel_gates(self, sums, decay_col, decay_rank, gate_col, gate_rank, decay_t, gate_t, dt_bias, a_log, decay, gate, n_tokens):
+    def channel_gates(self, sums, decay_col, decay_rank, gate_col, gate_rank, decay_t, gate_t, dt_bias, a_log, decay, gate, n_tokens,
+                      decay_w=None, gate_w=None):
         z = self._cols(sums, decay_col, decay_rank)[:n_tokens] @ decay_t.float() + dt_bias
         rate = torch.exp(a_log).repeat_interleave(decay_t.shape[1] // a_log.numel())
         decay[:n_tokens] = torch.exp(-rate * torch.nn.functional.softplus(z))
