@@ -5,7 +5,7 @@
 //   MODE 1  read with a bonus, decay, write:    o_t = (S + diag(u) k_t v_t^T)^T q_t;       S <- diag(a_t) S + k_t v_t^T
 //   MODE 2  delta rule with a decay a head:     S <- g_t S;  w = beta_t (v_t - S^T k_t);   S <- S + k_t w^T;   o_t = S^T q_t
 //           (q and k made unit vectors per head first: x / sqrt(sum x^2 + unit_eps))
-//   MODE 3  delta rule with a decay a channel:  S <- diag(a_t) S;  the rest as MODE 2, beta_t = sigmoid of its product's sums
+//   MODE 3  delta rule with a decay a channel:  S <- diag(a_t) S;  the rest as MODE 2, beta_t a number a head of its own
 //
 // Every column S[:, j] evolves by itself, so a block takes a (request, head, tile of columns) and walks the request's tokens of the
 // step in order; a column's dk numbers are spread over R lanes of a warp (KPT = 16 numbers a lane), the two dot products of a
@@ -19,7 +19,7 @@
 //
 // Beside it: token_shift (every projection's own blend of a token's input with the previous token's, the previous token of a
 // portion's first token coming from the slot), delta_gates (the delta rule's decay and write strength per head), channel_gates
-// (two low-rank maps at once: a decay per head and key channel, and the gate of the result) and head_norm_gate (every head's
+// (two low-rank maps and a sigmoid at once: a decay per head and key channel, the gate of the result, the write strength) and head_norm_gate (every head's
 // result divided by its root mean square, times a weight, times silu or sigmoid of a gate).
 #include "common.cuh"
 #include "mma_common.cuh"
@@ -46,7 +46,7 @@ struct Sums {  // columns off.. of float32 sums [parts, rows, width]
 };
 
 struct LinearStateParams {
-  Sums q, k, v, b;                                 // b: MODE 3, one number a head (before its sigmoid)
+  Sums q, k, v, b;                                 // b: MODE 3, one number a head
   const float* decay; int decay_width, decay_off;  // float32 rows: MODE 0/1/3 a number a (head, key channel); MODE 2 [g: H | beta: H]
   const float* bonus;                              // MODE 1: [H, dk]
   float* state;                                    // [slots, H, R * KPT, dv] in the layout above
@@ -294,8 +294,6 @@ template <int MODE>
 __device__ __forceinline__ void fetch_finish(const LinearStateParams& p, int cnt, int dk, int dkp, int tid, int n_thr, const TileRows& rows) {
   const bool unit = MODE >= 2 && p.unit_eps >= 0.f;
   const float qmul = unit ? 1.0f : p.q_scale;
-  if (MODE == 3)  // the thread's own numbers, as fetch_issue dealt them
-    for (int e = tid; e < cnt; e += n_thr) rows.b[e] = 1.0f / (1.0f + expf(-rows.b[e]));
   if (p.one_part && qmul != 1.0f) {  // the thread's own copies, as fetch_issue dealt them
     const int n_qk = cnt * dkp;
     if (p.vec4) {
@@ -451,14 +449,23 @@ __global__ void delta_gates_kernel(const Sums a, const Sums b, const float* __re
 
 // Two low-rank maps of one product's sums in one launch. Columns x0.off .. + R0 of the sums feed map 0, the decay of a delta rule
 // with a decay per key channel: out0[t, c] = exp(-exp(a_log[c / per]) * softplus(bias0[c] + sum_r w0[c, r] x0[t, r])); columns
-// x1.off .. + R1 feed map 1, out1[t, c] = sum_r w1[c, r] x1[t, r], the sums of the result's gate. All float32.
+// x1.off .. + R1 feed map 1, out1[t, c] = sum_r w1[c, r] x1[t, r], the sums of the result's gate. Beside them
+// beta[t, h] = sigmoid(xb[t, h]), the write strengths of H heads. All float32.
 struct ChannelGates {
-  Sums x0, x1;
-  int R0, R1, C0, C1, per;
+  Sums x0, x1, xb;
+  int R0, R1, C0, C1, per, H;
   const float* bias0; const float* a_log;
-  float* out0; float* out1;
+  float* out0; float* out1; float* beta;
   int n_tokens;
 };
+
+// beta of a block's tokens t0 .. t1: the first block of every row of blocks does it
+__device__ __forceinline__ void write_beta(const ChannelGates& p, int t0, int t1) {
+  for (int i = threadIdx.x; i < (t1 - t0) * p.H; i += blockDim.x) {
+    const int t = t0 + i / p.H, h = i % p.H;
+    p.beta[(size_t)t * p.H + h] = 1.0f / (1.0f + expf(-parts_sum(p.xb.p, p.xb.n, p.xb.stride, (size_t)t * p.xb.width + p.xb.off + h)));
+  }
+}
 
 __device__ __forceinline__ float channel_decay(float z, float a_log) {
   return expf(-expf(a_log) * (z > 20.0f ? z : log1pf(expf(z))));
@@ -479,10 +486,30 @@ __global__ void __launch_bounds__(128) channel_gates_kernel(const ChannelGates p
   float* low = sm_cg;
   float* quarter = sm_cg + (size_t)R * 8;
   const int t0 = blockIdx.y * 8;
-  for (int i = threadIdx.x; i < 8 * R; i += 128) {
-    const int tl = i / R, r = i - tl * R;
-    low[r * 8 + tl] = t0 + tl < p.n_tokens ? parts_sum(x.p, x.n, x.stride, (size_t)(t0 + tl) * x.width + x.off + r) : 0.f;
+  constexpr int U = 8;  // numbers a thread has in flight, part after part in the parts' order
+  for (int i0 = threadIdx.x; i0 < 8 * R; i0 += U * 128) {
+    float v[U];
+    size_t at[U];
+    bool ok[U];
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const int i = i0 + u * 128, tl = i / R, r = i - tl * R;
+      ok[u] = i < 8 * R && t0 + tl < p.n_tokens;
+      at[u] = (size_t)(t0 + tl) * x.width + x.off + r;
+      v[u] = 0.f;
+    }
+    for (int k = 0; k < x.n; ++k) {
+#pragma unroll
+      for (int u = 0; u < U; ++u)
+        if (ok[u]) v[u] += x.p[(size_t)k * x.stride + at[u]];
+    }
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const int i = i0 + u * 128, tl = i / R, r = i - tl * R;
+      if (i < 8 * R) low[r * 8 + tl] = v[u];
+    }
   }
+  if (blockIdx.x == 0) write_beta(p, t0, min(t0 + 8, p.n_tokens));
   __syncthreads();
   const int lane = threadIdx.x & 31, part = threadIdx.x >> 5;
   const int c = min(c0 + lane, C - 1);
@@ -531,13 +558,20 @@ __global__ void __launch_bounds__(CG_THREADS) channel_gates_mma_kernel(const Cha
   const bool quads = R % 8 == 0 && (reinterpret_cast<uintptr_t>(w) & 15u) == 0;
   for (int k0 = 0; k0 < R; k0 += CG_K) {
     if (k0 > 0) __syncthreads();  // everyone is done with the block before
-    for (int i = tid; i < CG_TOK * CG_K; i += CG_THREADS) {
-      const int t = i / CG_K, k = i % CG_K;
-      float v = 0.f;
-      if (t0 + t < p.n_tokens && k0 + k < R) v = parts_sum(x.p, x.n, x.stride, (size_t)(t0 + t) * x.width + x.off + k0 + k);
-      const bf16 h = __float2bfloat16_rn(v);
+    constexpr int U = CG_TOK * CG_K / CG_THREADS;  // numbers a thread has in flight
+    float v[U];
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const int i = tid + u * CG_THREADS, t = i / CG_K, k = i % CG_K;
+      v[u] = 0.f;
+      if (t0 + t < p.n_tokens && k0 + k < R) v[u] = x.p[(size_t)(t0 + t) * x.width + x.off + k0 + k];  // (one part)
+    }
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const int i = tid + u * CG_THREADS, t = i / CG_K, k = i % CG_K;
+      const bf16 h = __float2bfloat16_rn(v[u]);
       hi_s[t][k] = h;
-      lo_s[t][k] = __float2bfloat16_rn(v - __bfloat162float(h));
+      lo_s[t][k] = __float2bfloat16_rn(v[u] - __bfloat162float(h));
     }
     if (quads) {
       for (int i = tid; i < CG_COLS * (CG_K / 8); i += CG_THREADS) {
@@ -570,20 +604,37 @@ __global__ void __launch_bounds__(CG_THREADS) channel_gates_mma_kernel(const Cha
       }
     }
   }
+  if (blockIdx.x == 0) write_beta(p, t0, min(t0 + CG_TOK, p.n_tokens));
+  float* out = first ? p.out0 : p.out1;
 #pragma unroll
   for (int j = 0; j < 8; ++j) {
+    const int c = c0 + wn * 64 + j * 8 + 2 * (lane % 4);
+    if (c >= C) continue;
+    const bool two = c + 1 < C;
+    float b0 = 0.f, b1 = 0.f, r0 = 0.f, r1 = 0.f;
+    if (first) {
+      b0 = p.bias0[c];
+      r0 = expf(p.a_log[c / p.per]);
+      if (two) {
+        b1 = p.bias0[c + 1];
+        r1 = expf(p.a_log[(c + 1) / p.per]);
+      }
+    }
 #pragma unroll
-    for (int e = 0; e < 2; ++e) {
-      const int c = c0 + wn * 64 + j * 8 + 2 * (lane % 4) + e;
-      if (c >= C) continue;
-      const float b = first ? p.bias0[c] : 0.f, rate = first ? expf(p.a_log[c / p.per]) : 0.f;
-#pragma unroll
-      for (int half = 0; half < 2; ++half) {
-        const int t = t0 + wm * 16 + lane / 4 + half * 8;
-        if (t >= p.n_tokens) continue;
-        const float z = acc[j][2 * half + e] + b;
-        if (first) p.out0[(size_t)t * C + c] = expf(-rate * (z > 20.0f ? z : log1pf(expf(z))));
-        else p.out1[(size_t)t * C + c] = z;
+    for (int half = 0; half < 2; ++half) {
+      const int t = t0 + wm * 16 + lane / 4 + half * 8;
+      if (t >= p.n_tokens) continue;
+      float y0 = acc[j][2 * half] + b0, y1 = acc[j][2 * half + 1] + b1;
+      if (first) {
+        y0 = expf(-r0 * (y0 > 20.0f ? y0 : log1pf(expf(y0))));
+        y1 = expf(-r1 * (y1 > 20.0f ? y1 : log1pf(expf(y1))));
+      }
+      float* dst = out + (size_t)t * C + c;
+      if (two && (C & 1) == 0) {  // both numbers, on an 8-byte boundary
+        *reinterpret_cast<float2*>(dst) = make_float2(y0, y1);
+      } else {
+        dst[0] = y0;
+        if (two) dst[1] = y1;
       }
     }
   }
@@ -676,7 +727,7 @@ extern "C" int llm_linear_state(int mode, const float* q, int qn, long long qs, 
   LLM_REQUIRE(n_seqs > 0 && n_seqs <= 65535 && H > 0 && H <= 65535 && G > 0 && H % G == 0 && dv > 0, "linear_state: bad sizes");
   LLM_REQUIRE(llm_linear_state_lanes(dk) > 0, "linear_state: a key size of %d is not in 1..%d", dk, 32 * KPT);
   LLM_REQUIRE(mode >= 2 || G == H, "linear_state: only the delta rules share query/key heads");
-  LLM_REQUIRE(mode != 3 || (b && bn >= 1 && bo >= 0 && bo + H <= bw), "linear_state: the delta rule with a decay a channel needs the sums of beta");
+  LLM_REQUIRE(mode != 3 || (b && bn >= 1 && bo >= 0 && bo + H <= bw), "linear_state: the delta rule with a decay a channel needs beta");
   LLM_REQUIRE(q && k && v && decay && state && out && qn >= 1 && kn >= 1 && vn >= 1 && (mode != 1 || bonus), "linear_state: missing tensors");
   LLM_REQUIRE(qo + G * dk <= qw && ko + G * dk <= kw && vo + H * dv <= vw && decay_off + (mode == 2 ? 2 * H : H * dk) <= decay_width,
               "linear_state: columns outside their rows");
@@ -766,17 +817,20 @@ extern "C" int llm_delta_gates(const float* a, int an, long long as, int aw, int
 // x: float32 sums; columns x0.. (R0 of them) and x1.. (R1). wt0 [R0, C0], wt1 [R1, C1]: the maps transposed, in the engine's dtype;
 // w0, w1 (bfloat16 alone, or null): the maps as they are stored, for steps of more than 64 tokens on tensor cores.
 extern "C" int llm_channel_gates(const float* x, int xn, long long xs, int xw, int x0, int x1, int R0, int R1, const void* wt0, const void* wt1,
-                                 const void* w0, const void* w1, const float* bias0, const float* a_log, int C0, int C1, int per, float* out0, float* out1, int dtype,
-                                 int n_tokens, cudaStream_t stream) {
+                                 const void* w0, const void* w1, const float* bias0, const float* a_log, int C0, int C1, int per, float* out0, float* out1,
+                                 int xb, int H, float* beta, int dtype, int n_tokens, cudaStream_t stream) {
+  // beta [n_tokens, H] = sigmoid of columns xb .. + H
   if (n_tokens == 0) return LLM_OK;
   LLM_REQUIRE(n_tokens > 0 && x && xn >= 1 && wt0 && wt1 && bias0 && a_log && out0 && out1, "channel_gates: missing tensors");
   LLM_REQUIRE(R0 > 0 && R1 > 0 && C0 > 0 && C1 > 0 && per > 0 && C0 % per == 0, "channel_gates: bad sizes");
   LLM_REQUIRE(x0 >= 0 && x1 >= 0 && x0 + R0 <= xw && x1 + R1 <= xw, "channel_gates: columns outside the product");
   LLM_REQUIRE(dtype == LLM_F32 || dtype == LLM_BF16, "channel_gates: unknown dtype %d", dtype);
   ChannelGates p;
-  p.x0 = Sums{x, xn, (size_t)xs, xw, x0}; p.x1 = Sums{x, xn, (size_t)xs, xw, x1};
+  LLM_REQUIRE(beta && H > 0 && xb >= 0 && xb + H <= xw, "channel_gates: columns of the write strengths outside the product");
+  p.x0 = Sums{x, xn, (size_t)xs, xw, x0}; p.x1 = Sums{x, xn, (size_t)xs, xw, x1}; p.xb = Sums{x, xn, (size_t)xs, xw, xb};
+  p.H = H; p.beta = beta;
   p.R0 = R0; p.R1 = R1; p.C0 = C0; p.C1 = C1; p.per = per; p.bias0 = bias0; p.a_log = a_log; p.out0 = out0; p.out1 = out1; p.n_tokens = n_tokens;
-  if (dtype == LLM_BF16 && w0 && w1 && n_tokens > 64) {
+  if (dtype == LLM_BF16 && w0 && w1 && n_tokens > 64 && xn == 1) {
     dim3 tiles(ceil_div(C0, CG_COLS) + ceil_div(C1, CG_COLS), ceil_div(n_tokens, CG_TOK));
     LLM_REQUIRE(tiles.y <= 65535, "channel_gates: too many tokens in one step (%d)", n_tokens);
     launch_kernel(channel_gates_mma_kernel, tiles, CG_THREADS, 0, stream, p, (const bf16*)w0, (const bf16*)w1);

@@ -1387,7 +1387,7 @@ class CudaOps:
         "decay_write_read": S <- diag(a) S + k v^T, o = S^T q; "bonus_read_decay_write": o = (S + diag(bonus) k v^T)^T q, then
         S <- diag(a) S + k v^T; "delta": S <- g S, w = beta (v - S^T k), S <- S + k w^T, o = S^T q with q and k made unit vectors
         per head first (x / sqrt(sum x^2 + unit_eps); unit_eps < 0: as they are); "channel_delta": the same with S <- diag(a) S for its
-        first step and beta = the sigmoid of the float32 sums `beta` at column beta_off + head. q is multiplied by q_scale. q, k, v: float32 sums
+        first step and beta = the float32 sums `beta` at column beta_off + head. q is multiplied by q_scale. q, k, v: float32 sums
         ([parts, n, width] or [n, width]) read at column offsets, q and k with kv_heads heads of dk (head h reads head
         h // (heads / kv_heads)), v with heads of dv. decay: float32 rows; at decay_off a number per (head, key channel), or for
         "delta" [g: heads | beta: heads]; with decay_const a single row that holds for every token (decays that are constants
@@ -1454,22 +1454,23 @@ class CudaOps:
                                         _ptr(dt_bias), _ptr(out), c_int(n_tokens), c_int(H), _stream()), lib)
         return out
 
-    def channel_gates(self, sums, decay_col: int, decay_rank: int, gate_col: int, gate_rank: int, decay_t: torch.Tensor, gate_t: torch.Tensor,
-                      dt_bias: torch.Tensor, a_log: torch.Tensor, decay: torch.Tensor, gate: torch.Tensor, n_tokens: int,
+    def channel_gates(self, sums, decay_col: int, decay_rank: int, gate_col: int, gate_rank: int, beta_col: int, decay_t: torch.Tensor,
+                      gate_t: torch.Tensor, dt_bias: torch.Tensor, a_log: torch.Tensor, decay: torch.Tensor, gate: torch.Tensor,
+                      beta: torch.Tensor, n_tokens: int,
                       decay_w: Optional[torch.Tensor] = None, gate_w: Optional[torch.Tensor] = None) -> None:
-        """Two low-rank maps of the float32 `sums` [parts, n, width] in one launch: decay[t, c] = exp(-exp(a_log[c // per]) *
+        """What a delta rule with a decay a channel reads beside q, k and v, from the float32 `sums` [parts, n, width] in one launch: decay[t, c] = exp(-exp(a_log[c // per]) *
         softplus(dt_bias[c] + sum_r decay_t[r, c] * sums[t, decay_col + r])) with per = channels / len(a_log), and
-        gate[t, c] = sum_r gate_t[r, c] * sums[t, gate_col + r]. decay_t, gate_t [rank, channels]: the maps stored transposed;
-        decay, gate: float32 [n, channels]. decay_w, gate_w [channels, rank] (optional): the maps as they are stored; with them a
+        gate[t, c] = sum_r gate_t[r, c] * sums[t, gate_col + r]; beta[t, h] = sigmoid(sums[t, beta_col + h]). decay_t, gate_t [rank, channels]: the maps stored transposed;
+        decay, gate: float32 [n, channels], beta [n, len(a_log)]. decay_w, gate_w [channels, rank] (optional): the maps as they are stored; with them a
         bfloat16 step of more than 64 tokens runs on tensor cores."""
-        for t, name in ((dt_bias, "dt_bias"), (a_log, "a_log"), (decay, "decay"), (gate, "gate")):
+        for t, name in ((dt_bias, "dt_bias"), (a_log, "a_log"), (decay, "decay"), (gate, "gate"), (beta, "beta")):
             _need(t, "channel_gates." + name, torch.float32)
             assert t.is_contiguous()
         _need(decay_t, "channel_gates.decay_t"); _need(gate_t, "channel_gates.gate_t", decay_t.dtype)
         C0, C1 = decay_t.shape[1], gate_t.shape[1]
         assert decay_t.is_contiguous() and gate_t.is_contiguous() and decay_t.shape[0] == decay_rank and gate_t.shape[0] == gate_rank
         assert dt_bias.numel() == C0 and C0 % a_log.numel() == 0 and decay.shape[1] == C0 and gate.shape[1] == C1
-        assert decay.shape[0] >= n_tokens and gate.shape[0] >= n_tokens
+        assert decay.shape[0] >= n_tokens and gate.shape[0] >= n_tokens and beta.shape[0] >= n_tokens and beta.shape[1] == a_log.numel()
         mma = self.tensor_cores and decay_w is not None and gate_w is not None and decay_w.dtype == torch.bfloat16
         if mma:
             assert decay_w.is_contiguous() and gate_w.is_contiguous() and decay_w.shape == (C0, decay_rank) and gate_w.shape == (C1, gate_rank)
@@ -1478,7 +1479,8 @@ class CudaOps:
         self._check(lib.llm_channel_gates(p, parts, stride, width, c_int(decay_col), c_int(gate_col), c_int(decay_rank), c_int(gate_rank),
                                           _ptr(decay_t), _ptr(gate_t), _ptr(decay_w if mma else None), _ptr(gate_w if mma else None),
                                           _ptr(dt_bias), _ptr(a_log), c_int(C0), c_int(C1),
-                                          c_int(C0 // a_log.numel()), _ptr(decay), _ptr(gate), c_int(dtype_code(decay_t.dtype)), c_int(n_tokens),
+                                          c_int(C0 // a_log.numel()), _ptr(decay), _ptr(gate), c_int(beta_col), c_int(a_log.numel()),
+                                          _ptr(beta), c_int(dtype_code(decay_t.dtype)), c_int(n_tokens),
                                           _stream()), lib)
 
     def head_norm_gate(self, o: torch.Tensor, weight: torch.Tensor, gate, gate_off: int, eps: float, out: torch.Tensor, n_tokens: int,

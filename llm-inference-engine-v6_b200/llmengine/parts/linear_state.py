@@ -238,8 +238,8 @@ class GatedDelta(Mixer):
 
 class ChannelDelta(Mixer):
     """The delta rule with a decay per head and key channel (ChannelDeltaSpec). One product for everything that reads the mixer's
-    input, [q | k | v | W_a1 h | W_g1 h | beta]; the short convolutions; both low-rank maps (decays, gate) in one launch; the state
-    under the rule "channel_delta", which takes beta's sums as they come; the heads' norm with a sigmoid gate."""
+    input, [q | k | v | W_a1 h | W_g1 h | W_b h]; the short convolutions; both low-rank maps (decays, gate) and beta's sigmoid in one
+    launch; the state under the rule "channel_delta"; the heads' norm with a sigmoid gate."""
 
     def __init__(self, spec: ChannelDeltaSpec, env):
         super().__init__(spec, env)
@@ -284,11 +284,12 @@ class ChannelDelta(Mixer):
         ops.conv_silu(sums, 0, C, self.w_conv, None, cache.states["channel_delta.conv"], ctx, qkv)
         decay = ctx.ws.get("channel_delta.decay", (n, H * dk), torch.float32)
         gate = ctx.ws.get("channel_delta.gate", (n, H * dv), torch.float32)
-        ops.channel_gates(sums, a_off, s.decay_rank, g_off, s.gate_rank, self.w_a2_t, self.w_g2_t, self.dt_bias, self.a_log, decay, gate, n,
+        beta = ctx.ws.get("channel_delta.beta", (n, H), torch.float32)
+        ops.channel_gates(sums, a_off, s.decay_rank, g_off, s.gate_rank, b_off, self.w_a2_t, self.w_g2_t, self.dt_bias, self.a_log, decay, gate, beta, n,
                           decay_w=self.w_a2, gate_w=self.w_g2)
         o = ctx.ws.get("channel_delta.o", (n, H * dv), torch.float32)
         ops.linear_state("channel_delta", qkv, 0, qkv, G * dk, qkv, 2 * G * dk, decay, 0, None, cache.states["channel_delta.state"], ctx, o,
-                         H, G, dk, dv, q_scale=dk ** -0.5, unit_eps=s.unit_eps, beta=sums, beta_off=b_off)
+                         H, G, dk, dv, q_scale=dk ** -0.5, unit_eps=s.unit_eps, beta=beta)
         y = ctx.ws.get("channel_delta.y", (n, H * dv), dt)
         ops.head_norm_gate(o, self.norm_w, gate, 0, s.eps, y, n, H, dv, act="sigmoid")
         return add_into_stream_or_partials(ops, y, self.w_o, ctx, False, "channel_delta.delta")

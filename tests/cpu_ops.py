@@ -451,7 +451,7 @@ class CpuOps:
         Q = self._cols(q, q_off, kv_heads * dk).reshape(-1, kv_heads, dk) * q_scale
         K = self._cols(k, k_off, kv_heads * dk).reshape(-1, kv_heads, dk)
         V = self._cols(v, v_off, heads * dv).reshape(-1, heads, dv)
-        strength = torch.sigmoid(self._cols(beta, beta_off, heads)) if beta is not None else None
+        strength = self._cols(beta, beta_off, heads) if beta is not None else None
         if rule in ("delta", "channel_delta") and unit_eps >= 0:
             Q = Q / torch.sqrt((Q / q_scale).pow(2).sum(-1, keepdim=True) + unit_eps)
             K = K / torch.sqrt(K.pow(2).sum(-1, keepdim=True) + unit_eps)
@@ -516,12 +516,13 @@ class CpuOps:
         out[:n_tokens, H:] = torch.sigmoid(self._cols(b, b_off, H)[:n_tokens])
         return out
 
-    def channel_gates(self, sums, decay_col, decay_rank, gate_col, gate_rank, decay_t, gate_t, dt_bias, a_log, decay, gate, n_tokens,
+    def channel_gates(self, sums, decay_col, decay_rank, gate_col, gate_rank, beta_col, decay_t, gate_t, dt_bias, a_log, decay, gate, beta, n_tokens,
                       decay_w=None, gate_w=None):
         z = self._cols(sums, decay_col, decay_rank)[:n_tokens] @ decay_t.float() + dt_bias
         rate = torch.exp(a_log).repeat_interleave(decay_t.shape[1] // a_log.numel())
         decay[:n_tokens] = torch.exp(-rate * torch.nn.functional.softplus(z))
         gate[:n_tokens] = self._cols(sums, gate_col, gate_rank)[:n_tokens] @ gate_t.float()
+        beta[:n_tokens] = torch.sigmoid(self._cols(sums, beta_col, a_log.numel())[:n_tokens])
 
     def head_norm_gate(self, o, weight, gate, gate_off, eps, out, n_tokens, heads, dv, act="silu"):
         y = o[:n_tokens].view(n_tokens, heads, dv)

@@ -204,18 +204,22 @@ def latent_attention(h, w, p, m, eps, st, owner=None):
     T, pos0 = h.shape[0], st.get("n", 0)
     Wk, Wv = w[p + "uk"].view(H, dk, -1), w[p + "uv"].view(H, dv, -1)
     cs = st.setdefault("c", []) if owner is None else owner["c"]
+    K, V = st.setdefault("K", []), st.setdefault("V", [])   # this layer's keys and values of every latent so far, [H, *] each
     out = []
     for t in range(T):
         pos = pos0 + t
         if owner is None:
             cs.append(_r(rms(w[p + "dkv"] @ h[t], eps) * w[p + "dkv.norm"]))
         q = _r(w[p + "uq"] @ _r(rms(w[p + "dq"] @ h[t], eps) * w[p + "dq.norm"])).view(H, dk)
-        c = torch.stack(cs[first_visible(pos, m["mask"]["size"]):pos + 1])
+        K.append(Wk @ cs[pos])
+        V.append(Wv @ cs[pos])
+        lo = first_visible(pos, m["mask"]["size"])
+        k, v = torch.stack(K[lo:pos + 1]), torch.stack(V[lo:pos + 1])
         gate = sigmoid(w[p + "g"] @ h[t])
         heads = []
         for a in range(H):
-            pr = softmax_with_sink((c @ Wk[a].t()) @ q[a] * m["scale"], w[p + "sink"][a])
-            heads.append(pr @ (c @ Wv[a].t()) * gate[a])
+            pr = softmax_with_sink(k[:, a] @ q[a] * m["scale"], w[p + "sink"][a])
+            heads.append(pr @ v[:, a] * gate[a])
         out.append(torch.cat(heads))
     st["n"] = pos0 + T
     return _r(torch.stack(out)) @ w[p + "o"].t()
