@@ -542,7 +542,7 @@ __global__ void __launch_bounds__(128) channel_gates_kernel(const ChannelGates p
 // of 16 x 64 each; w0 [C0, R0], w1 [C1, R1] as the checkpoint stores them. The low-rank numbers enter as the sum of two bfloat16
 // numbers (the number rounded, and what the rounding left), a product each, so they count with about 16 bits of mantissa.
 constexpr int CG_TOK = 64, CG_COLS = 128, CG_K = 64, CG_LD = CG_K + 8, CG_THREADS = 256;
-__global__ void __launch_bounds__(CG_THREADS) channel_gates_mma_kernel(const ChannelGates p, const bf16* __restrict__ w0, const bf16* __restrict__ w1) {
+__global__ void __launch_bounds__(CG_THREADS, 3) channel_gates_mma_kernel(const ChannelGates p, const bf16* __restrict__ w0, const bf16* __restrict__ w1) {
   __shared__ __align__(16) bf16 hi_s[CG_TOK][CG_LD], lo_s[CG_TOK][CG_LD], w_s[CG_COLS][CG_LD];
   dep_launch();
   dep_wait();
