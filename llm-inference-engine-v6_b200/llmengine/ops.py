@@ -923,7 +923,8 @@ class CudaOps:
             if lib.llm_latent_attention_mma_supported(c_int(H), c_int(kv_rank), c_int(Dk - kv_rank)):
                 n_splits, split_keys, scratch = 1, 256, None
                 if batch.max_new_tokens == 1 and batch.n_tokens == batch.n_seqs:
-                    reach = min(batch.max_seq_len, window + 63) if window > 0 else batch.max_seq_len  # splits begin at the window's tile
+                    # splits begin at the tile of 64 that holds the window's first key, and a window's tiles are counted whole
+                    reach = min(batch.max_seq_len, (window + 126) // 64 * 64) if window > 0 else batch.max_seq_len
                     n_splits, split_keys = self._latent_split_policy(batch.n_seqs * -(-H // 32), reach)
                 if n_splits > 1:
                     floats = int(lib.llm_latent_attention_scratch_floats(c_int(batch.n_tokens), c_int(H), c_int(kv_rank), c_int(n_splits)))
