@@ -43,7 +43,7 @@ def config(vocab, width, eps, scale, pairs, logit_scale, layers, max_positions=5
 
 
 # ranks of the low-rank maps (decay, gate): no keys of config.json; make_tensors draws the maps with these first dimensions
-RANKS = {"za": {1: (5, 7), 4: (3, 2)}, "zb": {0: (24, 40), 3: (8, 16)}, "zc": {2: (1, 9)}}
+RANKS = {"za": {1: (5, 7), 4: (3, 2)}, "zb": {0: (32, 40), 3: (8, 16)}, "zc": {2: (1, 9)}}
 
 # A: nothing a multiple of 8; latent attention first and last, the last one on the first one's latents through a WIDER window; shared
 #    query/key heads in one delta layer, a single tap in the other; pages of 4
@@ -55,12 +55,12 @@ ZUDATAR_A = config(301, 72, 1e-5, 3.7, (53, 17, 5), 1.9, [
     layer("channel_delta", delta(3, 3, 18, 6, 1))])
 # B: sizes the tensor-core products and attention take (latents of 64 and 128, heads of 32 / 64 / 128); a borrower with a NARROWER
 #    window; a value size of its own; pages of 16
-ZUDATAR_B = config(512, 128, 1e-6, 8.0, (1021, 31, 127), 0.5, [
+ZUDATAR_B = config(512, 128, 1e-6, 8.0, (769, 31, 113), 0.6, [
     layer("channel_delta", delta(4, 2, 32, 64, 4), 256),
-    layer("attention", att(4, 2, 64, 0.125, 48, (32, 250000.0)), 384),
+    layer("attention", att(4, 2, 64, 0.15, 48, (24, 20000.0)), 384),
     layer("latent_attention", lat(6, 32, 48, 64, 40, 0.2, 40), 128),
     layer("channel_delta", delta(2, 2, 64, 32, 2)),
-    layer("latent_attention", lat(4, 64, 32, 64, 80, 0.125, 17, kv_from=2), 256),
+    layer("latent_attention", lat(4, 64, 32, 64, 72, 0.15, 17, kv_from=2), 256),
     layer("attention", att(5, 1, 32, 0.18, 24))])
 # C: one key/value head for five query heads, a window of one page, a window of a single key, two borrowers of one owner, a rank of
 #    one, one bucket, no rotation in one layer and a whole head's in another; pages of 8
