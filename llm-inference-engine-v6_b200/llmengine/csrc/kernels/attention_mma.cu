@@ -15,7 +15,7 @@
 // Options for mixers that want them, each off at 0 / null: keys and values of different sizes (HDK, HDV); `chunk`: a row at
 // position i reads only keys j with floor(j / chunk) == floor(i / chunk); `sink`: a float per query head whose exponential
 // is one more term of the softmax's denominator; `gate`: float32 partial sums whose sigmoid multiplies the result before
-// it is rounded (all three in the form without splits).
+// it is rounded (with splits, sink and gate are applied where the splits are merged).
 //
 // Formula: the reference's attention_f32 (src/kernels.cpp:413-474): kv head = q head / group,
 // score = (q . k) * scale applied after the dot, softmax, weighted sum of values.
@@ -375,28 +375,23 @@ int launch_plain(const AttnParams& p, int n_seqs, int max_new_tokens, cudaStream
   return 0;
 }
 
-template <int HD>
+template <int HD, int HDV = HD>
 int launch(const AttnParams& p, int n_seqs, int max_new_tokens, int n_tokens, bool split, cudaStream_t stream) {
-  constexpr int LD = HD + 8;
+  if (!split) return launch_plain<HD, HDV>(p, n_seqs, max_new_tokens, stream);
   const int g = p.nq / p.nkv;
   auto set_attr = [&](auto kernel, size_t smem) {
     if (smem > 48 * 1024) return cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) == cudaSuccess;
     return true;
   };
-  const size_t smem = (size_t)(M_TILE + 4 * N_TILE) * LD * sizeof(bf16);
+  const size_t smem = ((size_t)(M_TILE + 2 * N_TILE) * (HD + 8) + (size_t)2 * N_TILE * (HDV + 8)) * sizeof(bf16);
   const int tq_cap = M_TILE / g;
-  dim3 grid((max_new_tokens + tq_cap - 1) / tq_cap, n_seqs, p.nkv * (split ? p.n_splits : 1));
-  if (split) {
-    if (!set_attr(paged_attention_mma_kernel<HD, HD, true>, smem)) return 1;
-    launch_kernel(paged_attention_mma_kernel<HD, HD, true>, grid, THREADS, smem, stream, p);
-    const int items = n_tokens * p.nq;
-    launch_kernel(attention_combine_kernel<HD>, (items + 3) / 4, 128, 0, stream, (const float*)p.part_o, (const float*)p.part_ml,
-                  p.n_splits, p.part_stride_tokens, p.nq, p.out, p.ld_out, n_tokens, p.sink, p.gate, p.g_parts, p.g_pstride, p.g_width,
-                  p.g_off, p.g_head);
-  } else {
-    if (!set_attr(paged_attention_mma_kernel<HD, HD, false>, smem)) return 1;
-    launch_kernel(paged_attention_mma_kernel<HD, HD, false>, grid, THREADS, smem, stream, p);
-  }
+  dim3 grid((max_new_tokens + tq_cap - 1) / tq_cap, n_seqs, p.nkv * p.n_splits);
+  if (!set_attr(paged_attention_mma_kernel<HD, HDV, true>, smem)) return 1;
+  launch_kernel(paged_attention_mma_kernel<HD, HDV, true>, grid, THREADS, smem, stream, p);
+  const int items = n_tokens * p.nq;
+  launch_kernel(attention_combine_kernel<HDV>, (items + 3) / 4, 128, 0, stream, (const float*)p.part_o, (const float*)p.part_ml,
+                p.n_splits, p.part_stride_tokens, p.nq, p.out, p.ld_out, n_tokens, p.sink, p.gate, p.g_parts, p.g_pstride, p.g_width,
+                p.g_off, p.g_head);
   return 0;
 }
 
@@ -453,7 +448,7 @@ extern "C" int llm_paged_attention_mma(const void* q, long long ld_q, const void
 
 // The same kernel with its options: keys of dk and values of dv numbers a head (each 32, 64 or 128), chunks, a sink per query
 // head, a gate given as float32 partial sums [g_parts, tokens, g_width] read at columns g_off + head * dv + d. A (request,
-// key/value head, tile of query rows) is one CTA that walks the keys it may see; steps of single tokens with dk == dv may cut
+// key/value head, tile of query rows) is one CTA that walks the keys it may see; steps of single tokens may cut
 // the key range into n_splits pieces of split_keys keys (scratch: llm_attention_mma_scratch_floats), counted from the start of
 // the token's chunk, with sink and gate applied where the pieces are merged.
 extern "C" int llm_gated_attention_mma_supported(int nq, int nkv, int dk, int dv, long long ld_q, long long ld_out) {
@@ -470,8 +465,8 @@ extern "C" int llm_gated_attention_mma(const void* q, long long ld_q, const void
                                        long long g_pstride, int g_width, int g_off, int g_head, int n_tokens, int n_splits, int split_keys,
                                        float* scratch, cudaStream_t stream) {
   if (n_seqs == 0 || max_new_tokens == 0) return LLM_OK;
-  LLM_REQUIRE(n_splits >= 1 && (n_splits == 1 || (dk == dv && max_new_tokens == 1 && split_keys > 0 && split_keys % N_TILE == 0 && scratch != nullptr)),
-              "gated_attention_mma: splits are for single tokens with keys and values of one size, split_keys %% 64 == 0, and need scratch");
+  LLM_REQUIRE(n_splits >= 1 && (n_splits == 1 || (max_new_tokens == 1 && split_keys > 0 && split_keys % N_TILE == 0 && scratch != nullptr)),
+              "gated_attention_mma: splits are for single tokens, split_keys %% 64 == 0, and need scratch");
   LLM_REQUIRE((long long)nkv * n_splits <= 65535, "gated_attention_mma: too many splits for the grid");
   LLM_REQUIRE(llm_gated_attention_mma_supported(nq, nkv, dk, dv, ld_q, ld_out), "gated_attention_mma: geometry not supported (nq=%d nkv=%d dk=%d dv=%d)", nq, nkv, dk, dv);
   LLM_REQUIRE(page_size > 0 && max_blocks > 0 && window >= 0 && chunk >= 0 && max_new_tokens > 0, "gated_attention_mma: bad sizes");
@@ -488,15 +483,8 @@ extern "C" int llm_gated_attention_mma(const void* q, long long ld_q, const void
   p.n_splits = n_splits; p.split_keys = split_keys; p.part_stride_tokens = n_tokens;
   p.part_o = scratch; p.part_ml = scratch ? scratch + (size_t)n_splits * n_tokens * nq * dv : nullptr;
   int rc = 1;
-  if (n_splits > 1) {  // the key range of every (request, key/value head) in pieces side by side, merged by a second kernel
-    if (dk == 32) rc = launch<32>(p, n_seqs, max_new_tokens, n_tokens, true, stream);
-    else if (dk == 64) rc = launch<64>(p, n_seqs, max_new_tokens, n_tokens, true, stream);
-    else rc = launch<128>(p, n_seqs, max_new_tokens, n_tokens, true, stream);
-    LLM_REQUIRE(rc == 0, "gated_attention_mma: cannot raise the shared memory limit");
-    LLM_CHECK_LAUNCH("gated_attention_mma");
-    return LLM_OK;
-  }
-#define LLM_GATED(K, V) if (dk == K && dv == V) rc = launch_plain<K, V>(p, n_seqs, max_new_tokens, stream)
+  // n_splits > 1: the key range of every (request, key/value head) in pieces side by side, merged by a second kernel
+#define LLM_GATED(K, V) if (dk == K && dv == V) rc = launch<K, V>(p, n_seqs, max_new_tokens, n_tokens, n_splits > 1, stream)
   LLM_GATED(32, 32); LLM_GATED(32, 64); LLM_GATED(32, 128);
   LLM_GATED(64, 32); LLM_GATED(64, 64); LLM_GATED(64, 128);
   LLM_GATED(128, 32); LLM_GATED(128, 64); LLM_GATED(128, 128);

@@ -483,11 +483,11 @@ extern "C" int llm_token_gate(const void* z, const void* table, long long ld_tab
   return LLM_OK;
 }
 
-// h += a (+ b), each float32 [parts, rows, dim] partial sums added in index order, a before b; then
-// copy (may be null) = h in the engine's dtype: the stream as the operand of a product.
+// h += a (+ b), each float32 [parts, rows, dim] partial sums added in index order, a before b (bias: a row [dim] that goes with a,
+// an output projection's bias); then copy (may be null) = h in the engine's dtype: the stream as the operand of a product.
 template <typename T>
 __global__ void stream_add_kernel(float* __restrict__ h, const float* __restrict__ a, int na, size_t sa, const float* __restrict__ b,
-                                  int nb, size_t sb, T* __restrict__ copy, size_t total) {
+                                  int nb, size_t sb, T* __restrict__ copy, size_t total, const float* __restrict__ bias, int dim) {
   dep_launch();
   dep_wait();
   const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
@@ -498,6 +498,7 @@ __global__ void stream_add_kernel(float* __restrict__ h, const float* __restrict
     for (int p = 1; p < na; ++p) d += a[(size_t)p * sa + i];
     x += d;
   }
+  if (bias) x += bias[i % dim];
   if (b) {
     float d = b[i];
     for (int p = 1; p < nb; ++p) d += b[(size_t)p * sb + i];
@@ -508,14 +509,17 @@ __global__ void stream_add_kernel(float* __restrict__ h, const float* __restrict
 }
 
 extern "C" int llm_stream_add(float* h, const float* a, int na, long long sa, const float* b, int nb, long long sb, void* copy,
-                              int copy_dtype, long long total, cudaStream_t stream) {
+                              int copy_dtype, long long total, const float* bias, int dim, cudaStream_t stream) {
   if (total == 0) return LLM_OK;
+  LLM_REQUIRE(bias == nullptr || dim > 0, "stream_add: a bias needs the row's size");
   LLM_REQUIRE(total > 0 && (a == nullptr || na >= 1) && (b == nullptr || nb >= 1), "stream_add: bad sizes");
   const int blocks = ceil_div(total, 256);
   if (copy_dtype == LLM_F32)
-    launch_kernel(stream_add_kernel<float>, blocks, 256, 0, stream, h, a, na, (size_t)sa, b, nb, (size_t)sb, (float*)copy, (size_t)total);
+    launch_kernel(stream_add_kernel<float>, blocks, 256, 0, stream, h, a, na, (size_t)sa, b, nb, (size_t)sb, (float*)copy, (size_t)total,
+                  bias, dim);
   else if (copy_dtype == LLM_BF16)
-    launch_kernel(stream_add_kernel<bf16>, blocks, 256, 0, stream, h, a, na, (size_t)sa, b, nb, (size_t)sb, (bf16*)copy, (size_t)total);
+    launch_kernel(stream_add_kernel<bf16>, blocks, 256, 0, stream, h, a, na, (size_t)sa, b, nb, (size_t)sb, (bf16*)copy, (size_t)total,
+                  bias, dim);
   else
     LLM_REQUIRE(false, "stream_add: unknown dtype %d", copy_dtype);
   LLM_CHECK_LAUNCH("stream_add");

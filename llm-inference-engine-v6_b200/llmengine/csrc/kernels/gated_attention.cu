@@ -9,6 +9,8 @@
 //              token's page. Keys have dk numbers a head, values dv. Options (QkvOptions, qkv_prep_after_kernel): a bias on the q and
 //              k columns; pairs of neighbours (2i, 2i + 1) turning together; every head divided by its root mean square behind the
 //              rotation; values that are the keys before any norm and rotation (the product then has no value columns).
+//              qkv_prep_row_kernel keeps a token's whole row in shared memory and takes biases on q, k and v, a short causal convolution
+//              of all three, either norm, either kind of pairs and a number a position that multiplies the queries.
 //   attention  one warp a (token, query head): keys lo..pos of the request through its block table, lo = the later of the
 //              window's and the chunk's start (a chunk is [c * size, (c + 1) * size) in absolute positions); softmax in float32
 //              whose denominator also holds exp(sink[head]) (optional: a learned term of the denominator alone); the result times
@@ -262,6 +264,168 @@ __global__ void __launch_bounds__(PREP_WARPS * 32)
   }
 }
 
+// A block a token, with the token's whole [q | k] row in shared memory:
+//   x[c] = bias[c] + sum_j conv_w[j, c] * u_(t - taps + 1 + j)[c]   (taps 0: x = bias + u), u the product's sums of the request's tokens;
+//          inputs before the step's portion come from the request's slot of conv_state [slots, taps - 1, C], zero when it starts
+//   norms of q and k (a head or the projection at once), rotation of either kind of pairs, q times q_mul[position]
+// `single`: every request of the step brings one token, so this block is the only one that reads the request's slot, and it renews
+// it: the same thread reads and then writes a channel's inputs. Longer portions renew the slots in a kernel behind this one.
+// A thread takes V neighbouring numbers at a time (V 4: 16-byte loads; every offset and row is then a multiple of four numbers).
+struct QkvRow {
+  const float* parts; int n_parts; size_t pstride; int width;
+  int H, G, dk, dv, rot_dims;
+  const float* bias;                                      // [q | k] or [q | k | v] numbers (bias_n of them), or null
+  int bias_n;
+  const float* conv_w; int taps; float* conv_state; int single;
+  const float* wq; const float* wk; int norm_wide; float eps;
+  const float* cos_t; const float* sin_t; int neighbours;
+  const float* q_mul;                                     // a number a position, or null
+  const int* positions; const int* token_seq; const int* seq_qoff; const int* seq_slot; const int* block_table;
+  int max_blocks, page_size;
+  long long ld_q;
+};
+
+template <int V>
+__device__ __forceinline__ void load_f32(float (&x)[V], const float* p) {
+  if constexpr (V == 4) {
+    const float4 t = *reinterpret_cast<const float4*>(p);
+    x[0] = t.x; x[1] = t.y; x[2] = t.z; x[3] = t.w;
+  } else {
+#pragma unroll
+    for (int e = 0; e < V; ++e) x[e] = p[e];
+  }
+}
+template <int V>
+__device__ __forceinline__ void store_f32(float* p, const float (&x)[V]) {
+  if constexpr (V == 4) *reinterpret_cast<float4*>(p) = make_float4(x[0], x[1], x[2], x[3]);
+  else
+#pragma unroll
+    for (int e = 0; e < V; ++e) p[e] = x[e];
+}
+template <int V>
+__device__ __forceinline__ void store_as(float* p, const float (&x)[V]) { store_f32<V>(p, x); }
+template <int V>
+__device__ __forceinline__ void store_as(bf16* p, const float (&x)[V]) {
+  if constexpr (V == 4) {
+    const __nv_bfloat162 a = __floats2bfloat162_rn(x[0], x[1]), b = __floats2bfloat162_rn(x[2], x[3]);
+    uint2 u;
+    u.x = *reinterpret_cast<const uint32_t*>(&a);
+    u.y = *reinterpret_cast<const uint32_t*>(&b);
+    *reinterpret_cast<uint2*>(p) = u;
+  } else {
+#pragma unroll
+    for (int e = 0; e < V; ++e) p[e] = __float2bfloat16_rn(x[e]);
+  }
+}
+template <int V>
+__device__ __forceinline__ void parts_sum_n(float (&s)[V], const float* p, int n_parts, size_t pstride) {  // parts in index order
+  load_f32<V>(s, p);
+#pragma unroll 4
+  for (int k = 1; k < n_parts; ++k) {
+    float t[V];
+    load_f32<V>(t, p + (size_t)k * pstride);
+#pragma unroll
+    for (int e = 0; e < V; ++e) s[e] += t[e];
+  }
+}
+
+template <typename T, int V>
+__global__ void __launch_bounds__(512) qkv_prep_row_kernel(const QkvRow p, T* __restrict__ q_out, T* __restrict__ kcache, T* __restrict__ vcache) {
+  extern __shared__ __align__(16) float row_sh[];  // [(H + G) * dk] numbers, then a factor a head
+  __shared__ float red[33];
+  dep_launch();
+  dep_wait();
+  const int tok = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n_warps = blockDim.x >> 5;
+  const int dk = p.dk, dv = p.dv, nq = p.H * dk, nqk = (p.H + p.G) * dk, C = nqk + p.G * dv;
+  float* inv_sh = row_sh + nqk;
+  const int pos = p.positions[tok], seq = p.token_seq[tok];
+  const int page = p.block_table[(size_t)seq * p.max_blocks + pos / p.page_size], in_page = pos % p.page_size;
+  const int first = p.seq_qoff[seq];
+  float* st = p.taps > 1 ? p.conv_state + (size_t)p.seq_slot[seq] * (p.taps - 1) * C : nullptr;
+  float ssq = 0.f, ssk = 0.f;
+  for (int c = threadIdx.x * V; c < C; c += blockDim.x * V) {
+    float x[V];
+    parts_sum_n<V>(x, p.parts + (size_t)tok * p.width + c, p.n_parts, p.pstride);
+    if (p.taps > 0) {
+      float acc[V], w[V], u[V];
+#pragma unroll
+      for (int e = 0; e < V; ++e) acc[e] = 0.f;
+      for (int j = 0; j < p.taps - 1; ++j) {
+        const int src = tok - (p.taps - 1) + j;
+        if (src >= first) parts_sum_n<V>(u, p.parts + (size_t)src * p.width + c, p.n_parts, p.pstride);
+        else load_f32<V>(u, st + (size_t)((p.taps - 1) + (src - first)) * C + c);  // src - first in [-(taps - 1), -1]
+        load_f32<V>(w, p.conv_w + (size_t)j * C + c);
+        if (p.single && j > 0) store_f32<V>(st + (size_t)(j - 1) * C + c, u);  // (src < first: u came from row j)
+#pragma unroll
+        for (int e = 0; e < V; ++e) acc[e] = fmaf(w[e], u[e], acc[e]);
+      }
+      if (p.single && p.taps > 1) store_f32<V>(st + (size_t)(p.taps - 2) * C + c, x);
+      load_f32<V>(w, p.conv_w + (size_t)(p.taps - 1) * C + c);
+#pragma unroll
+      for (int e = 0; e < V; ++e) x[e] = fmaf(w[e], x[e], acc[e]);
+    }
+    if (c < p.bias_n) {
+      float b[V];
+      load_f32<V>(b, p.bias + c);
+#pragma unroll
+      for (int e = 0; e < V; ++e) x[e] += b[e];
+    }
+    if (c < nqk) {
+      store_f32<V>(row_sh + c, x);
+      float s = 0.f;
+#pragma unroll
+      for (int e = 0; e < V; ++e) s += x[e] * x[e];
+      if (c < nq) ssq += s;
+      else ssk += s;
+    } else if (vcache) {
+      const int i = c - nqk, g = i / dv, d = i - g * dv;
+      store_as<V>(vcache + (((size_t)page * p.G + g) * p.page_size + in_page) * dv + d, x);
+    }
+  }
+  if (p.norm_wide) {  // one statistic a projection
+    const float inv_q = p.wq ? 1.0f / sqrtf(block_sum(ssq, red) / (float)nq + p.eps) : 1.0f;
+    const float inv_k = (p.wk && p.G > 0) ? 1.0f / sqrtf(block_sum(ssk, red) / (float)(nqk - nq) + p.eps) : 1.0f;
+    for (int h = threadIdx.x; h < p.H + p.G; h += blockDim.x) inv_sh[h] = h < p.H ? inv_q : inv_k;
+  } else if (p.wq || p.wk) {
+    __syncthreads();  // the row is complete
+    for (int h = warp; h < p.H + p.G; h += n_warps) {
+      float ss = 0.f;
+      for (int d = lane; d < dk; d += 32) ss += row_sh[h * dk + d] * row_sh[h * dk + d];
+      ss = warp_sum(ss);
+      if (lane == 0) inv_sh[h] = 1.0f / sqrtf(ss / (float)dk + p.eps);
+    }
+  }
+  __syncthreads();
+  const int half = p.rot_dims / 2;
+  const float* cs = p.cos_t ? p.cos_t + (size_t)pos * half : nullptr;
+  const float* sn = p.sin_t ? p.sin_t + (size_t)pos * half : nullptr;
+  const float q_mul = p.q_mul ? p.q_mul[pos] : 1.0f;
+  for (int c = threadIdx.x * V; c < (kcache ? nqk : nq); c += blockDim.x * V) {
+    const int head = c / dk, d0 = c - head * dk;
+    const bool is_q = head < p.H;
+    const float* row = row_sh + head * dk;
+    const float* w = is_q ? p.wq : p.wk;
+    if (w && p.norm_wide) w += (size_t)(is_q ? head : head - p.H) * dk;  // a weight a number of the projection
+    const float inv = w ? inv_sh[head] : 1.0f;
+    auto at = [&](int d) { return w ? row[d] * inv * w[d] : row[d]; };
+    float x[V];
+#pragma unroll
+    for (int e = 0; e < V; ++e) {
+      const int d = d0 + e;
+      x[e] = at(d);
+      if (d < p.rot_dims) {
+        const bool second = p.neighbours ? (d & 1) : d >= half;
+        const int i = p.neighbours ? d >> 1 : (second ? d - half : d);
+        const float y = at(p.neighbours ? d ^ 1 : (second ? d - half : d + half));
+        x[e] = second ? x[e] * cs[i] + y * sn[i] : x[e] * cs[i] - y * sn[i];
+      }
+      if (is_q) x[e] *= q_mul;
+    }
+    if (is_q) store_as<V>(q_out + (size_t)tok * p.ld_q + c, x);
+    else store_as<V>(kcache + (((size_t)page * p.G + (head - p.H)) * p.page_size + in_page) * dk + d0, x);
+  }
+}
+
 constexpr int WARPS = 4;
 constexpr int MAX_HD = 512;
 
@@ -413,6 +577,50 @@ extern "C" int llm_qkv_prep(const float* parts, int n_parts, long long pstride, 
   else LLM_REQUIRE(false, "qkv_prep: unknown dtype %d", dtype);
 #undef LLM_PREP
   LLM_CHECK_LAUNCH("qkv_prep");
+  return LLM_OK;
+}
+
+// qkv_prep with a token's row in shared memory (qkv_prep_row_kernel). bias: bias_n = (H + G) * dk numbers, or G * dv more, or null.
+// conv_w [taps, C] float32 with C = (H + G) * dk + G * dv, conv_state [slots, taps - 1, C]; single: every request of the step brings one
+// token, and the slots are renewed here (else by llm_conv_state behind this call). q_mul: a float32 number a position.
+extern "C" int llm_qkv_prep_row(const float* parts, int n_parts, long long pstride, int width, int H, int G, int dk, int dv, int rot_dims,
+                                const float* bias, int bias_n, const float* conv_w, int taps, float* conv_state, int single, const float* wq,
+                                const float* wk, int norm_wide, float eps, const float* cos_t, const float* sin_t, int neighbours,
+                                const float* q_mul, const int* positions, const int* token_seq, const int* seq_qoff, const int* seq_slot,
+                                const int* block_table, int max_blocks, void* q_out, long long ld_q, void* kcache, void* vcache, int page_size,
+                                int dtype, int n_tokens, cudaStream_t stream) {
+  if (n_tokens == 0) return LLM_OK;
+  const long long nqk = (long long)(H + G) * dk, C = nqk + (long long)G * dv;
+  LLM_REQUIRE(n_tokens > 0 && n_parts >= 1 && H > 0 && G >= 0 && dk > 0 && dv > 0 && taps >= 0 && taps <= 16, "qkv_prep: bad sizes (taps %d, at most 16)", taps);
+  LLM_REQUIRE(G > 0 || kcache == nullptr, "qkv_prep: a product without keys and values writes none");
+  LLM_REQUIRE((kcache == nullptr) == (vcache == nullptr), "qkv_prep: keys and values are written together");
+  LLM_REQUIRE(rot_dims >= 0 && rot_dims % 2 == 0 && rot_dims <= dk, "qkv_prep: %d rotated dimensions do not fit a head of %d", rot_dims, dk);
+  LLM_REQUIRE(rot_dims == 0 || (cos_t && sin_t), "qkv_prep: rotation tables missing");
+  LLM_REQUIRE(C <= width, "qkv_prep: columns outside the product");
+  LLM_REQUIRE(bias ? (bias_n == nqk || bias_n == C) : bias_n == 0, "qkv_prep: a bias of %d numbers", bias_n);
+  LLM_REQUIRE(taps == 0 || (conv_w && (taps == 1 || conv_state)), "qkv_prep: the convolution needs weights and the slots' inputs");
+  LLM_REQUIRE(page_size > 0 && max_blocks > 0, "qkv_prep: bad page_size/max_blocks");
+  const size_t smem = ((size_t)nqk + H + G) * sizeof(float);
+  LLM_REQUIRE(smem <= 200 * 1024, "qkv_prep: a token's queries and keys (%lld numbers) exceed one block's shared memory", nqk);
+  QkvRow p{parts, n_parts, (size_t)pstride, width, H, G, dk, dv, rot_dims, bias, bias_n, conv_w, taps, conv_state, single, wq, wk, norm_wide, eps,
+           cos_t, sin_t, neighbours, q_mul, positions, token_seq, seq_qoff, seq_slot, block_table, max_blocks, page_size, ld_q};
+  auto quads = [](const void* q) { return ((uintptr_t)q & 15u) == 0; };
+  const bool vec = dk % 4 == 0 && dv % 4 == 0 && width % 4 == 0 && pstride % 4 == 0 && ld_q % 4 == 0 && quads(parts) && quads(bias) && quads(conv_w) &&
+                   quads(conv_state) && quads(q_out) && quads(kcache) && quads(vcache);
+  const int groups = (int)(vec ? C / 4 : C);
+  // few tokens: a number of threads that takes a token's row in one go; many tokens: several blocks a multiprocessor
+  const int threads = n_tokens >= 512 ? min(256, ceil_div(groups, 32) * 32) : min(512, ceil_div(groups, 32) * 32);
+#define LLM_PREP_ROW(T, V)                                                                                                               \
+  LLM_REQUIRE(smem <= 40 * 1024 || cudaFuncSetAttribute(qkv_prep_row_kernel<T, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024) == \
+              cudaSuccess, "qkv_prep: cannot raise the shared memory limit");                                                               \
+  launch_kernel(qkv_prep_row_kernel<T, V>, n_tokens, threads, smem, stream, p, (T*)q_out, (T*)kcache, (T*)vcache)
+  if (dtype == LLM_F32 && vec) { LLM_PREP_ROW(float, 4); }
+  else if (dtype == LLM_F32) { LLM_PREP_ROW(float, 1); }
+  else if (dtype == LLM_BF16 && vec) { LLM_PREP_ROW(bf16, 4); }
+  else if (dtype == LLM_BF16) { LLM_PREP_ROW(bf16, 1); }
+  else LLM_REQUIRE(false, "qkv_prep: unknown dtype %d", dtype);
+#undef LLM_PREP_ROW
+  LLM_CHECK_LAUNCH("qkv_prep_row");
   return LLM_OK;
 }
 

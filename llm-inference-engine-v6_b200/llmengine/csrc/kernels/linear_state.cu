@@ -20,7 +20,8 @@
 // Beside it: token_shift (every projection's own blend of a token's input with the previous token's, the previous token of a
 // portion's first token coming from the slot), delta_gates (the delta rule's decay and write strength per head), channel_gates
 // (two low-rank maps and a sigmoid at once: a decay per head and key channel, the gate of the result, the write strength) and head_norm_gate (every head's
-// result divided by its root mean square, times a weight, times silu or sigmoid of a gate).
+// result divided by its root mean square, times a weight, times silu or sigmoid of a gate; wide heads, or all heads as one, a block a
+// row) and silu_sums (activated projections for portions, whose tiles then arrive as they are).
 #include "common.cuh"
 #include "mma_common.cuh"
 
@@ -33,6 +34,7 @@ constexpr int LS_THREADS = 128;   // threads that hold the state, at most: fewer
 constexpr int LS_FETCHERS = 128;  // threads behind them that fetch the tiles of tokens ahead
 constexpr int LS_BLOCK = LS_THREADS + LS_FETCHERS;
 constexpr int LS_BUFFERS = 3;    // tiles in shared memory: walked, landing, issued
+constexpr int WIDE_NORM_FROM = 512;  // rows of more numbers are normed by a block each
 constexpr size_t LS_SMEM = 112 * 1024;  // of the tiles, at most (portions)
 
 __device__ __forceinline__ float parts_sum(const float* __restrict__ p, int n_parts, size_t pstride, size_t i) {
@@ -54,6 +56,7 @@ struct LinearStateParams {
   float* out;                                      // [tokens, H * dv]
   int H, G, dk, dv, R, tile;
   float q_scale, unit_eps;
+  int silu;      // q, k and v are silu of the sums
   int walkers;   // threads of a block that hold the state (a multiple of 32 and of R); LS_FETCHERS more fetch
   int one_part;  // every product comes in one part
   int vec4;      // every row and column offset is a multiple of four numbers on a 16-byte boundary
@@ -172,11 +175,14 @@ __device__ __forceinline__ void copy16_async(float* smem_dst, const float* gmem_
 __device__ __forceinline__ void copies_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
 __device__ __forceinline__ void copies_wait_but_last() { asm volatile("cp.async.wait_group 1;" ::: "memory"); }
 
+__device__ __forceinline__ float silu_f(float v) { return v / (1.0f + expf(-v)); }
+
 // A tile's rows into shared memory by the n_thr fetching threads (thread `tid` of them), in two steps so that two tiles can be
 // on their way while a third is walked. fetch_issue: every thread takes elements of the whole tile in turn. Products in one
 // part (a prompt's portion) are copied asynchronously (16 bytes a copy where every address allows it), no registers held, and
 // the copies of a tile are one group. Products in several parts (few tokens, K cut) go through registers, a few elements at a
-// time, the parts added in their order. fetch_finish, once the tile's group has landed: the thread scales its own queries; the
+// time, the parts added in their order (and silu applied, where the rule reads activated projections). fetch_finish, once the tile's
+// group has landed: the thread activates its own copies and scales its own queries; the
 // delta rule's unit norms need a token's whole row, so the fetchers meet (barrier 1 is theirs alone) and a warp a token
 // scales what was stored.
 template <int MODE>
@@ -261,8 +267,8 @@ __device__ __forceinline__ void fetch_issue(const LinearStateParams& p, size_t r
     for (int x = 0; x < U; ++x) {
       const int e = e0 + x * n_thr;
       if (e < n_qk) {
-        rows.q[e] = qv[x] * qmul;
-        rows.k[e] = kv[x];
+        rows.q[e] = (p.silu ? silu_f(qv[x]) : qv[x]) * qmul;
+        rows.k[e] = p.silu ? silu_f(kv[x]) : kv[x];
         if (MODE != 2) rows.a[e] = av[x];
       }
     }
@@ -282,7 +288,7 @@ __device__ __forceinline__ void fetch_issue(const LinearStateParams& p, size_t r
     }
 #pragma unroll
     for (int x = 0; x < U; ++x)
-      if (e0 + x * n_thr < n_v) rows.v[e0 + x * n_thr] = vv[x];
+      if (e0 + x * n_thr < n_v) rows.v[e0 + x * n_thr] = p.silu ? silu_f(vv[x]) : vv[x];
   }
   if (MODE == 2)
     for (int e = tid; e < 2 * cnt; e += n_thr) rows.a[e] = p.decay[(row0 + (e >> 1)) * p.decay_width + p.decay_off + (e & 1) * p.H + head];
@@ -291,11 +297,21 @@ __device__ __forceinline__ void fetch_issue(const LinearStateParams& p, size_t r
 }
 
 template <int MODE>
-__device__ __forceinline__ void fetch_finish(const LinearStateParams& p, int cnt, int dk, int dkp, int tid, int n_thr, const TileRows& rows) {
+__device__ __forceinline__ void fetch_finish(const LinearStateParams& p, int cnt, int dk, int dkp, int dv, int tid, int n_thr, const TileRows& rows) {
   const bool unit = MODE >= 2 && p.unit_eps >= 0.f;
   const float qmul = unit ? 1.0f : p.q_scale;
-  if (p.one_part && qmul != 1.0f) {  // the thread's own copies, as fetch_issue dealt them
-    const int n_qk = cnt * dkp;
+  const int n_qk = cnt * dkp;
+  if (p.one_part && p.silu) {  // the thread's own copies, as fetch_issue dealt them (a group of four numbers or one)
+    const int n_v = cnt * dv, V = p.vec4 ? 4 : 1;
+    for (int e = tid * V; e < n_qk; e += n_thr * V)
+      for (int i = e; i < e + V; ++i) {
+        rows.q[i] = silu_f(rows.q[i]);
+        rows.k[i] = silu_f(rows.k[i]);
+      }
+    for (int e = tid * V; e < n_v; e += n_thr * V)
+      for (int i = e; i < e + V; ++i) rows.v[i] = silu_f(rows.v[i]);
+  }
+  if (p.one_part && qmul != 1.0f) {
     if (p.vec4) {
       for (int e = tid; e < (n_qk >> 2); e += n_thr) {
         float4 t = *reinterpret_cast<float4*>(rows.q + 4 * e);
@@ -365,7 +381,7 @@ __global__ void __launch_bounds__(LS_BLOCK, FEW ? 2 : 1) linear_state_kernel(con
     copies_commit();
   };
   auto finish = [&](int i) {
-    if (i < n_tiles) fetch_finish<MODE>(p, min(tile, n_tok - i * tile), dk, dkp, ftid, n_fetch, rows_of(i));
+    if (i < n_tiles) fetch_finish<MODE>(p, min(tile, n_tok - i * tile), dk, dkp, dv, ftid, n_fetch, rows_of(i));
   };
 
   float* st = p.state + ((size_t)p.seq_slot[seq] * p.H + head) * (size_t)dkp * dv;
@@ -668,6 +684,51 @@ __global__ void __launch_bounds__(128)
   }
 }
 
+// The same for wide rows (all heads normed together): a block a (token, head), its numbers in the threads' turns, then block_sum.
+template <typename T>
+__global__ void __launch_bounds__(1024)
+    wide_norm_gate_kernel(const float* __restrict__ o, const float* __restrict__ weight, int weight_per_head, const Sums gate, float eps,
+                          T* __restrict__ out, int H, int dv, int sigmoid) {
+  __shared__ float red[33];
+  dep_launch();
+  dep_wait();
+  const size_t item = blockIdx.x, tok = item / H;
+  const int head = (int)(item - tok * H);
+  const float* row = o + item * dv;
+  float ss = 0.f;
+  for (int d = threadIdx.x; d < dv; d += blockDim.x) ss = fmaf(row[d], row[d], ss);
+  const float inv = 1.0f / sqrtf(block_sum(ss, red) / (float)dv + eps);
+  for (int d = threadIdx.x; d < dv; d += blockDim.x) {
+    float v = row[d] * inv * weight[weight_per_head ? (size_t)head * dv + d : d];
+    if (gate.p) {
+      const float g = parts_sum(gate.p, gate.n, gate.stride, tok * gate.width + gate.off + (size_t)head * dv + d);
+      v *= (sigmoid ? 1.0f : g) / (1.0f + expf(-g));
+    }
+    out[item * dv + d] = from_f32<T>(v);
+  }
+}
+
+// out[t, c] = silu(columns off .. + C of the sums), float32: four neighbouring numbers a thread
+template <int V>
+__global__ void silu_sums_kernel(const Sums x, int C, float* __restrict__ out, size_t total) {
+  dep_launch();
+  dep_wait();
+  const size_t i = ((size_t)blockIdx.x * blockDim.x + threadIdx.x) * V;
+  if (i >= total) return;
+  const size_t tok = i / C;
+  const size_t src = tok * x.width + x.off + (i - tok * C);
+  if constexpr (V == 4) {
+    float4 s = *reinterpret_cast<const float4*>(x.p + src);
+    for (int k = 1; k < x.n; ++k) {
+      const float4 t = *reinterpret_cast<const float4*>(x.p + (size_t)k * x.stride + src);
+      s.x += t.x; s.y += t.y; s.z += t.z; s.w += t.w;
+    }
+    *reinterpret_cast<float4*>(out + i) = make_float4(silu_f(s.x), silu_f(s.y), silu_f(s.z), silu_f(s.w));
+  } else {
+    out[i] = silu_f(parts_sum(x.p, x.n, x.stride, src));
+  }
+}
+
 int device_sms() {
   static int n = 0;
   if (n == 0) {
@@ -720,8 +781,9 @@ extern "C" int llm_linear_state(int mode, const float* q, int qn, long long qs, 
                                 int ko, const float* v, int vn, long long vs, int vw, int vo, const float* b, int bn, long long bs, int bw,
                                 int bo, const float* decay, int decay_width, int decay_off, const float* bonus, float* state, const int* seq_qoff, const int* seq_ntok,
                                 const int* seq_slot, float* out, int n_tokens, int n_seqs, int H, int G, int dk, int dv, float q_scale,
-                                float unit_eps, int decay_const, cudaStream_t stream) {
-  // decay_const: `decay` is one row that holds for every token (decays that are constants of the model)
+                                float unit_eps, int decay_const, int silu, cudaStream_t stream) {
+  // decay_const: `decay` is one row that holds for every token (decays that are constants of the model); silu: q, k and v are silu of
+  // the sums (before the query's scale)
   if (n_seqs == 0) return LLM_OK;
   LLM_REQUIRE(mode >= 0 && mode <= 3, "linear_state: unknown update rule %d", mode);
   LLM_REQUIRE(n_seqs > 0 && n_seqs <= 65535 && H > 0 && H <= 65535 && G > 0 && H % G == 0 && dv > 0, "linear_state: bad sizes");
@@ -736,7 +798,7 @@ extern "C" int llm_linear_state(int mode, const float* q, int qn, long long qs, 
   p.b = Sums{b, bn, (size_t)bs, bw, bo};
   p.decay = decay; p.decay_width = decay_const ? 0 : decay_width; p.decay_off = decay_off; p.bonus = bonus; p.state = state;
   p.seq_qoff = seq_qoff; p.seq_ntok = seq_ntok; p.seq_slot = seq_slot; p.out = out;
-  p.H = H; p.G = G; p.dk = dk; p.dv = dv; p.R = lanes_for(dk); p.q_scale = q_scale; p.unit_eps = unit_eps;
+  p.H = H; p.G = G; p.dk = dk; p.dv = dv; p.R = lanes_for(dk); p.q_scale = q_scale; p.unit_eps = unit_eps; p.silu = silu;
   const int dkp = p.R * KPT;
   const int a_stride = mode == 2 ? 2 : dkp;
   auto smem_for = [&](int tile) {  // as the kernel lays a buffer out
@@ -854,14 +916,37 @@ extern "C" int llm_head_norm_gate(const float* o, const float* weight, int weigh
   LLM_REQUIRE(n_tokens > 0 && H > 0 && dv > 0 && o && weight && out, "head_norm_gate: bad arguments");
   LLM_REQUIRE(gate == nullptr || (gn >= 1 && go >= 0 && go + H * dv <= gw), "head_norm_gate: gate columns outside the product");
   const Sums g{gate, gn, (size_t)gs, gw, go};
+  LLM_REQUIRE(dtype == LLM_F32 || dtype == LLM_BF16, "head_norm_gate: unknown dtype %d", dtype);
+  if (dv > WIDE_NORM_FROM) {  // a block a row; the threads' number depends on the row's size alone, and with it the order of the sum
+    const int threads = min(1024, ceil_div(dv, 128) * 32);
+    const long long rows = (long long)n_tokens * H;
+    LLM_REQUIRE(rows <= 0x7fffffffLL, "head_norm_gate: too many rows");
+    if (dtype == LLM_F32)
+      launch_kernel(wide_norm_gate_kernel<float>, (int)rows, threads, 0, stream, o, weight, weight_per_head, g, eps, (float*)out, H, dv, sigmoid);
+    else
+      launch_kernel(wide_norm_gate_kernel<bf16>, (int)rows, threads, 0, stream, o, weight, weight_per_head, g, eps, (bf16*)out, H, dv, sigmoid);
+    LLM_CHECK_LAUNCH("head_norm_gate");
+    return LLM_OK;
+  }
   const int blocks = ceil_div((long long)n_tokens * H, 4);
   if (dtype == LLM_F32)
     launch_kernel(head_norm_gate_kernel<float>, blocks, 128, 0, stream, o, weight, weight_per_head, g, eps, (float*)out, n_tokens, H, dv, sigmoid);
-  else if (dtype == LLM_BF16)
-    launch_kernel(head_norm_gate_kernel<bf16>, blocks, 128, 0, stream, o, weight, weight_per_head, g, eps, (bf16*)out, n_tokens, H, dv, sigmoid);
   else
-    LLM_REQUIRE(false, "head_norm_gate: unknown dtype %d", dtype);
+    launch_kernel(head_norm_gate_kernel<bf16>, blocks, 128, 0, stream, o, weight, weight_per_head, g, eps, (bf16*)out, n_tokens, H, dv, sigmoid);
   LLM_CHECK_LAUNCH("head_norm_gate");
+  return LLM_OK;
+}
+
+extern "C" int llm_silu_sums(const float* x, int xn, long long xs, int xw, int xo, int C, float* out, int n_tokens, cudaStream_t stream) {
+  if (n_tokens == 0) return LLM_OK;
+  LLM_REQUIRE(n_tokens > 0 && C > 0 && x && out && xn >= 1 && xo >= 0 && (long long)xo + C <= xw, "silu_sums: bad arguments");
+  const Sums s{x, xn, (size_t)xs, xw, xo};
+  const long long total = (long long)n_tokens * C;
+  if (C % 4 == 0 && xw % 4 == 0 && xo % 4 == 0 && xs % 4 == 0 && (((uintptr_t)x | (uintptr_t)out) & 15u) == 0)
+    launch_kernel(silu_sums_kernel<4>, ceil_div(total / 4, 256), 256, 0, stream, s, C, out, (size_t)total);
+  else
+    launch_kernel(silu_sums_kernel<1>, ceil_div(total, 256), 256, 0, stream, s, C, out, (size_t)total);
+  LLM_CHECK_LAUNCH("silu_sums");
   return LLM_OK;
 }
 

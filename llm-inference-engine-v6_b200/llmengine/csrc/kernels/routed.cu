@@ -8,7 +8,8 @@
 //             one expert (the last tile of an expert is padded with -1); tile_expert[i] = -1 for unused tiles
 //   product   for every tile: rows of a (picked by pair / a_div) times the expert's matrix; the result row
 //             is written at the pair's index, so no inverse permutation is needed. Epilogue: the exact
-//             (erf) gelu, or the pair's weight
+//             (erf) gelu, the pair's weight, or the square of relu of the sum times the pair's weight (a weight that
+//             multiplies what an expert reads: its first matrix is linear)
 //   combine   out[t] = sum over the token's choices, in index order
 #include "common.cuh"
 
@@ -236,7 +237,7 @@ __global__ void group_kernel(const int* __restrict__ idx, int n_pairs, int E, in
 
 constexpr int RP_WARPS = 4, RP_ROWS = 8;  // rows of a tile of the CUDA-core product
 
-// epilogue 0: exact gelu; 1: times share[pair]; 2: w holds 2 N rows, row 2 n a gate and row 2 n + 1 its up row:
+// epilogue 0: exact gelu; 1: times share[pair] (null: as it is); 3: max(share[pair] * sum, 0)^2 (null: 1); 2: w holds 2 N rows, row 2 n a gate and row 2 n + 1 its up row:
 // out[p, n] = gated_value(gate, up) with the activation (act, p0, p1) of common.cuh: silu(gate) * up, or both sides limited
 template <typename TA, typename TO>
 __global__ void __launch_bounds__(RP_WARPS * 32)
@@ -295,7 +296,13 @@ __global__ void __launch_bounds__(RP_WARPS * 32)
       if (i == lane) { v = acc[i]; p = pair[i]; }
     if (p >= 0) {
       if (epilogue == 0) v = 0.5f * v * (1.0f + erff(v * 0.70710678118654752440f));
-      else if (epilogue == 1) v *= share[p];
+      else if (epilogue != 2) {
+        if (share) v *= share[p];
+        if (epilogue == 3) {
+          v = fmaxf(v, 0.f);
+          v *= v;
+        }
+      }
       out[(size_t)p * ldo + n] = from_f32<TO>(v);
     }
   }
@@ -392,7 +399,7 @@ extern "C" int llm_routed_product(const void* a, long long lda, int a_div, const
   // act, p0, p1: the activation of epilogue 2 (0: silu; 2: both sides limited by p0, slope p1)
   if (max_tiles == 0) return LLM_OK;
   LLM_REQUIRE(N > 0 && K > 0 && a_div > 0 && max_tiles > 0 && max_tiles <= 65535, "routed_product: bad sizes");
-  LLM_REQUIRE(epilogue == 0 || (epilogue == 1 && share) || (epilogue == 2 && N % 2 == 0), "routed_product: unknown epilogue %d", epilogue);
+  LLM_REQUIRE(epilogue == 0 || epilogue == 1 || epilogue == 3 || (epilogue == 2 && N % 2 == 0), "routed_product: unknown epilogue %d", epilogue);
   LLM_REQUIRE(act >= 0 && act <= 2, "routed_product: unknown activation %d", act);
   const long long ws = (long long)N * K;
   if (epilogue == 2) N /= 2;  // outputs: one for every (gate, up) pair of rows

@@ -5,7 +5,8 @@
 // pair / a_div of the operand), its B rows are 64 rows of the expert's matrix [N, K]. K is walked in blocks of 64
 // with cp.async through a ring of three stages in shared memory; four warps of 16 rows each (m16n8k16). Every output row is
 // written at its pair's own index; a row's sum depends on K alone, not on the rest of its tile.
-// Epilogue 0: the exact (erf) gelu, bfloat16 out; 1: times the pair's router weight, float32 out; 2: the matrix holds a gate
+// Epilogue 0: the exact (erf) gelu, bfloat16 out; 1: times the pair's router weight (if there is one), float32 out; 3: the square of
+// relu of the sum times the pair's router weight, bfloat16 out (a weight on what an expert reads); 2: the matrix holds a gate
 // row and its up row in turn (an even number of rows), out[p, n / 2] = act(gate, up) (silu(gate) * up, or both sides limited: common.cuh), bfloat16 out.
 // heads_product_mma: the same tile loop for a product per head over all tokens (the key and value maps of latent attention).
 #include "common.cuh"
@@ -96,7 +97,7 @@ __global__ void __launch_bounds__(RM_THREADS * WM)
     for (int half = 0; half < 2; ++half) {
       const int pair = rows_s[(warp_m * WM + i) * 16 + lane / 4 + half * 8];
       if (pair < 0) continue;
-      const float sc = EPI == 1 ? share[pair] : 1.0f;
+      const float sc = ((EPI == 1 || EPI == 3) && share) ? share[pair] : 1.0f;
       TO* dst = out + (size_t)pair * ldo;
 #pragma unroll
       for (int j = 0; j < RM_COLS / 8; ++j) {
@@ -114,6 +115,10 @@ __global__ void __launch_bounds__(RM_THREADS * WM)
           }
           if (EPI == 0) v = 0.5f * v * (1.0f + erff(v * 0.70710678118654752440f));
           else v *= sc;
+          if (EPI == 3) {
+            v = fmaxf(v, 0.f);
+            v *= v;
+          }
           dst[n] = from_f32<TO>(v);
         }
       }
@@ -191,7 +196,7 @@ __global__ void __launch_bounds__(RM_THREADS)
   for (int half = 0; half < 2; ++half) {
     const int pair = rows_s[lane / 4 + half * 8];
     if (pair < 0) continue;
-    const float sc = EPI == 1 ? share[pair] : 1.0f;
+    const float sc = ((EPI == 1 || EPI == 3) && share) ? share[pair] : 1.0f;
     TO* dst = out + (size_t)pair * ldo;
 #pragma unroll
     for (int j = 0; j < 2; ++j) {
@@ -209,6 +214,10 @@ __global__ void __launch_bounds__(RM_THREADS)
         }
         if (EPI == 0) v = 0.5f * v * (1.0f + erff(v * 0.70710678118654752440f));
         else v *= sc;
+        if (EPI == 3) {
+          v = fmaxf(v, 0.f);
+          v *= v;
+        }
         dst[n] = from_f32<TO>(v);
       }
     }
@@ -333,11 +342,12 @@ extern "C" int llm_routed_product_mma(const void* a, long long lda, int a_div, c
   LLM_REQUIRE(llm_routed_product_mma_supported(a, lda, w, K), "routed_product_mma: operands must be 16-byte aligned with K and the row stride multiples of 8");
   LLM_REQUIRE(N > 0 && a_div > 0 && max_tiles > 0 && max_tiles <= 65535, "routed_product_mma: bad sizes");
   LLM_REQUIRE(tile == RS_ROWS || tile == RM_ROWS || tile == 2 * RM_ROWS, "routed_product_mma: tiles of %d rows (16, 64 or 128)", tile);
-  LLM_REQUIRE(epilogue == 0 || (epilogue == 1 && share) || (epilogue == 2 && N % 2 == 0), "routed_product_mma: unknown epilogue %d", epilogue);
+  LLM_REQUIRE(epilogue == 0 || epilogue == 1 || epilogue == 3 || (epilogue == 2 && N % 2 == 0), "routed_product_mma: unknown epilogue %d", epilogue);
   if (tile == RS_ROWS) {
     static bool raised_few = false;
     if (!raised_few) {
       LLM_REQUIRE(cudaFuncSetAttribute(routed_product_mma_few_kernel<bf16, 0>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)RS_SMEM) == cudaSuccess &&
+                  cudaFuncSetAttribute(routed_product_mma_few_kernel<bf16, 3>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)RS_SMEM) == cudaSuccess &&
                   cudaFuncSetAttribute(routed_product_mma_few_kernel<bf16, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)RS_SMEM) == cudaSuccess &&
                   cudaFuncSetAttribute(routed_product_mma_few_kernel<float, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)RS_SMEM) == cudaSuccess,
                   "routed_product_mma: cannot raise the shared memory limit");
@@ -350,6 +360,9 @@ extern "C" int llm_routed_product_mma(const void* a, long long lda, int a_div, c
                     N, K, tile_expert, tile_rows, (bf16*)out, ldo, share, act, p0, p1);
     else if (epilogue == 2)
       launch_kernel(routed_product_mma_few_kernel<bf16, 2>, grid_few, RM_THREADS, RS_SMEM, stream, (const bf16*)a, lda, a_div, (const bf16*)w, wsf,
+                    N, K, tile_expert, tile_rows, (bf16*)out, ldo, share, act, p0, p1);
+    else if (epilogue == 3)
+      launch_kernel(routed_product_mma_few_kernel<bf16, 3>, grid_few, RM_THREADS, RS_SMEM, stream, (const bf16*)a, lda, a_div, (const bf16*)w, wsf,
                     N, K, tile_expert, tile_rows, (bf16*)out, ldo, share, act, p0, p1);
     else
       launch_kernel(routed_product_mma_few_kernel<float, 1>, grid_few, RM_THREADS, RS_SMEM, stream, (const bf16*)a, lda, a_div, (const bf16*)w, wsf,
@@ -367,6 +380,9 @@ extern "C" int llm_routed_product_mma(const void* a, long long lda, int a_div, c
   else if (epilogue == 2)
     rc = wm == 2 ? launch_routed<bf16, 2, 2>(grid, stream, a, lda, a_div, w, ws, N, K, tile_expert, tile_rows, out, ldo, share, act, p0, p1)
                  : launch_routed<bf16, 2, 1>(grid, stream, a, lda, a_div, w, ws, N, K, tile_expert, tile_rows, out, ldo, share, act, p0, p1);
+  else if (epilogue == 3)
+    rc = wm == 2 ? launch_routed<bf16, 3, 2>(grid, stream, a, lda, a_div, w, ws, N, K, tile_expert, tile_rows, out, ldo, share, act, p0, p1)
+                 : launch_routed<bf16, 3, 1>(grid, stream, a, lda, a_div, w, ws, N, K, tile_expert, tile_rows, out, ldo, share, act, p0, p1);
   else
     rc = wm == 2 ? launch_routed<float, 1, 2>(grid, stream, a, lda, a_div, w, ws, N, K, tile_expert, tile_rows, out, ldo, share, act, p0, p1)
                  : launch_routed<float, 1, 1>(grid, stream, a, lda, a_div, w, ws, N, K, tile_expert, tile_rows, out, ldo, share, act, p0, p1);

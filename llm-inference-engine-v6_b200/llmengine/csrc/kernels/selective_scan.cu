@@ -403,6 +403,17 @@ __global__ void scan_carry_kernel(const float* __restrict__ a_log, float* __rest
 
 }  // namespace
 
+// The slots' convolution inputs after a step: the last K - 1 inputs of every request, from the step's tokens and the old slot.
+extern "C" int llm_conv_state(const float* parts, int n_parts, long long pstride, int width, int x_off, int C, int K, float* conv_state,
+                              const int* seq_qoff, const int* seq_ntok, const int* seq_slot, int n_seqs, cudaStream_t stream) {
+  if (K <= 1 || n_seqs == 0) return LLM_OK;  // a single tap keeps nothing
+  LLM_REQUIRE(n_seqs > 0 && n_parts >= 1 && C > 0 && K <= MAX_TAPS && x_off >= 0 && x_off + C <= width, "conv_state: bad sizes (taps %d, at most %d)", K, MAX_TAPS);
+  launch_kernel(conv_state_kernel, ceil_div((long long)n_seqs * C, 256), 256, 0, stream, parts, n_parts, (size_t)pstride, width, x_off, C, K,
+                conv_state, seq_qoff, seq_ntok, seq_slot, n_seqs);
+  LLM_CHECK_LAUNCH("conv_state");
+  return LLM_OK;
+}
+
 extern "C" int llm_conv_silu(const float* parts, int n_parts, long long pstride, int width, int x_off, int C, int K, const void* w,
                              const float* bias, float* conv_state, const int* token_seq, const int* seq_qoff, const int* seq_ntok,
                              const int* seq_slot, void* out, int dtype, int n_tokens, int n_seqs, cudaStream_t stream) {
@@ -430,12 +441,7 @@ extern "C" int llm_conv_silu(const float* parts, int n_parts, long long pstride,
   else
     LLM_REQUIRE(false, "conv_silu: unknown dtype %d", dtype);
   LLM_CHECK_LAUNCH("conv_silu");
-  if (K > 1) {
-    launch_kernel(conv_state_kernel, ceil_div((long long)n_seqs * C, 256), 256, 0, stream, parts, n_parts, (size_t)pstride, width, x_off, C, K,
-                  conv_state, seq_qoff, seq_ntok, seq_slot, n_seqs);
-    LLM_CHECK_LAUNCH("conv_state");
-  }
-  return LLM_OK;
+  return llm_conv_state(parts, n_parts, pstride, width, x_off, C, K, conv_state, seq_qoff, seq_ntok, seq_slot, n_seqs, stream);
 }
 
 // dt[t, c] = out_act(bias[c] + sum_r wt[r, c] * in_act(proj[t, r])): the step-size map of the selective scan (in_act 0, out_act 0) and

@@ -83,6 +83,10 @@ class StepContext:
         # layer with value mixing hands to the layers after it); tensors of the workspace, so their addresses stay fixed
         self.shared: Dict[str, object] = {}
         self.embedding_cache = None  # parts.base.LayerCache of the embedding's own state, if it keeps any
+        # set by a block while it runs a mixer whose output projection's bias it adds itself, where it adds the mixer's sums to the
+        # stream: such a mixer leaves the float32 vector in delta_bias
+        self.takes_delta_bias = False
+        self.delta_bias = None
         self.takes_delta_pairs = False  # set by a block while it runs a feed-forward whose two branches' sums it adds itself
 
 

@@ -1,2 +1,2 @@
 """Architectures: each module registers one name of config.json `architectures` (or `architecture`)."""
-from . import llama, selinex, sogutar, vapelix, zudatar, zulopel  # noqa: F401
+from . import kasarax, llama, selinex, sogutar, vapelix, zudatar, zulopel  # noqa: F401

@@ -801,8 +801,9 @@ class CudaOps:
 
     # ------------------------------------------------------------------ stream and token side input
     def stream_add(self, h: torch.Tensor, a: Optional[torch.Tensor], b: Optional[torch.Tensor] = None,
-                   copy: Optional[torch.Tensor] = None, n_rows: Optional[int] = None) -> torch.Tensor:
-        """h[:n] += a (+ b): float32 [n, dim] or [parts, n, dim] partial sums added in index order, a before b;
+                   copy: Optional[torch.Tensor] = None, n_rows: Optional[int] = None, bias: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """h[:n] += a (+ b): float32 [n, dim] or [parts, n, dim] partial sums added in index order, a before b; bias (float32 [dim],
+        optional) is added to every row as well;
         copy[:n] (optional, float32 or bfloat16) = the new h, the stream as an operand of a product."""
         _need(h, "stream_add.h", torch.float32)
         n = h.shape[0] if n_rows is None else n_rows
@@ -820,8 +821,12 @@ class CudaOps:
             _need(copy, "stream_add.copy")
             assert copy.is_contiguous() and copy.shape[-1] == h.shape[-1] and copy.shape[0] >= n
             code = dtype_code(copy.dtype)
+        if bias is not None:
+            _need(bias, "stream_add.bias", torch.float32)
+            assert bias.is_contiguous() and bias.numel() == h.shape[-1]
         assert h.is_contiguous()
-        self._check(lib.llm_stream_add(_ptr(h), *args, _ptr(copy), c_int(code), c_longlong(n * h.shape[-1]), _stream()), lib)
+        self._check(lib.llm_stream_add(_ptr(h), *args, _ptr(copy), c_int(code), c_longlong(n * h.shape[-1]), _ptr(bias), c_int(h.shape[-1]),
+                                       _stream()), lib)
         return h
 
     def token_gate(self, z: torch.Tensor, table: torch.Tensor, col0: int, ids: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
@@ -992,7 +997,7 @@ class CudaOps:
         self._check(lib.llm_route(_ptr(x), c_longlong(x.stride(0)), _ptr(w), _ptr(bias), c_int(n), c_int(D), c_int(E), c_int(top),
                                   _ptr(idx), _ptr(share), c_int(dtype_code(x.dtype)), _stream()), lib)
 
-    ROUTED_EPILOGUES = {"gelu": 0, "share": 1, "silu_pairs": 2, "gated_pairs": 2}
+    ROUTED_EPILOGUES = {"gelu": 0, "share": 1, "silu_pairs": 2, "gated_pairs": 2, "relu_squared": 3}
 
     def route_grouped(self, x: torch.Tensor, w: torch.Tensor, correction: Optional[torch.Tensor], top: int, groups: int, keep: int,
                       norm_eps: float, idx: torch.Tensor, share: torch.Tensor, score: str = "softmax", group_top: int = 1,
@@ -1045,7 +1050,8 @@ class CudaOps:
     def routed_product(self, a: torch.Tensor, a_div: int, w: torch.Tensor, tile_expert: torch.Tensor, tile_rows: torch.Tensor,
                        out: torch.Tensor, epilogue: str, share: Optional[torch.Tensor] = None, act="silu") -> torch.Tensor:
         """For every pair p of every tile (expert e): out[p, :] = epi(w[e] a[p // a_div, :]); w [E, N, K]. epilogue "gelu":
-        the exact (erf) gelu; "share": times share[p] (float32, flat); "silu_pairs": w holds a gate row and its up row in turn
+        the exact (erf) gelu; "share": times share[p] (float32, flat; None: as it is); "relu_squared": max(share[p] * z, 0)^2 (share None: 1),
+        which for a share on what the expert reads is the same as on its linear product; "silu_pairs": w holds a gate row and its up row in turn
         ([E, 2 F, K]) and out[p, f] = silu(gate_f) * up_f ([pairs, F]); "gated_pairs": the same rows with the activation `act`
         of a gated feed-forward (ACTIVATIONS; ("clamped_swish", limit, slope) limits both sides)."""
         _need(a, "routed_product.a"); _need(w, "routed_product.w", a.dtype); _need(out, "routed_product.out")
@@ -1054,7 +1060,7 @@ class CudaOps:
         assert w.is_contiguous() and a.shape[1] == K and out.shape[1] == (N // 2 if pairs else N)
         assert not pairs or N % 2 == 0
         act_args = self._act_args(act if epilogue == "gated_pairs" else "silu")
-        if epilogue == "share":
+        if share is not None:
             _need(share, "routed_product.share", torch.float32)
         if a.dtype == torch.bfloat16 and self.tensor_cores and tile_rows.shape[1] != self.routed_tile_rows():
             lib = self.lib("tensorcore")  # tiles made for the tensor-core kernel (64 or 128 rows)
@@ -1137,30 +1143,36 @@ class CudaOps:
                  block_table: torch.Tensor, q_out: torch.Tensor, kcache: Optional[torch.Tensor], vcache: Optional[torch.Tensor],
                  mix_role: int = 0, mix_weight: Optional[torch.Tensor] = None, v_first: Optional[torch.Tensor] = None,
                  norm_wide: bool = False, bias: Optional[torch.Tensor] = None, neighbours: bool = False, unit_rms: bool = False,
-                 keys_as_values: bool = False) -> None:
+                 keys_as_values: bool = False, conv: Optional[torch.Tensor] = None, conv_state: Optional[torch.Tensor] = None,
+                 q_mul: Optional[torch.Tensor] = None) -> None:
         """From the float32 sums `parts` [p, n, width] of a product whose columns begin with [q: heads * dk | k: kv_heads * dk |
         v: kv_heads * dv] (kv_heads 0: queries alone, nothing to write): RMS norm of every query and key head with the weights
         q_norm / k_norm [dk] (None: no norm), or with norm_wide ONE RMS norm over all query heads' numbers together with q_norm
         [heads * dk] and one over all key heads' with k_norm [kv_heads * dk]; rotation
         of the first 2 * cos.shape[1] numbers of each head (half-split pairs) at the token's position, q into q_out
         [n, heads * dk], k and v into the token's page of kcache [pages, kv_heads, page, dk] / vcache [.., dv] (None: no write).
-        bias (float32 [(heads + kv_heads) * dk]) is added to the q and k columns first; neighbours: the rotation's pairs are (2i, 2i + 1);
+        bias (float32 [(heads + kv_heads) * dk], or kv_heads * dv more) is added to the q and k (and v) columns first; neighbours: the rotation's pairs are (2i, 2i + 1);
         unit_rms: every head is divided by its root mean square after the rotation; keys_as_values: the product has no v columns, the
         values are its k columns (with their bias, before norm and rotation; dv == dk).
         mix_role 1: the values are also left in v_first (float32 [n, kv_heads * dv]); 2: v <- (1 - m) v + m v_first before
-        the write, m = mix_weight (a float32 scalar on the device)."""
+        the write, m = mix_weight (a float32 scalar on the device).
+        conv (float32 [taps, C], C = (heads + kv_heads) * dk + kv_heads * dv): before the bias every column c becomes sum_j conv[j, c] *
+        (the column's sum of the request's token taps - 1 - j before), the inputs before the step's portion taken from conv_state
+        [slots, taps - 1, C] (float32) at the request's slot, which afterwards holds the request's last taps - 1 inputs. q_mul
+        (float32, a number a position): the finished queries are multiplied by it."""
         _need(parts, "qkv_prep.parts", torch.float32); _need(q_out, "qkv_prep.q")
         assert parts.dim() == 3 and parts.is_contiguous()
         n = batch.n_tokens
         rot_dims = 0 if cos is None else 2 * cos.shape[1]
         for t, name in ((q_norm, "q_norm"), (k_norm, "k_norm"), (cos, "cos"), (sin, "sin"), (mix_weight, "mix_weight"), (v_first, "v_first"),
-                        (bias, "bias")):
+                        (bias, "bias"), (conv, "conv"), (conv_state, "conv_state"), (q_mul, "q_mul")):
             if t is not None:
                 _need(t, "qkv_prep." + name, torch.float32)
                 assert t.is_contiguous()
         wide = (heads, kv_heads) if norm_wide else (1, 1)
         assert (q_norm is None or q_norm.numel() == wide[0] * dk) and (k_norm is None or kv_heads == 0 or k_norm.numel() == wide[1] * dk)
-        assert bias is None or bias.numel() == (heads + kv_heads) * dk
+        n_qk, channels = (heads + kv_heads) * dk, (heads + kv_heads) * dk + kv_heads * dv
+        assert bias is None or bias.numel() in (n_qk, channels)
         page = 1
         if kcache is not None:
             _need(kcache, "qkv_prep.kcache", q_out.dtype); _need(vcache, "qkv_prep.vcache", q_out.dtype)
@@ -1170,6 +1182,26 @@ class CudaOps:
         if v_first is not None:
             assert v_first.shape[0] >= n and v_first.shape[1] == kv_heads * dv
         lib = self.lib()
+        if conv is not None or q_mul is not None or (norm_wide and neighbours) or (bias is not None and (bias.numel() != n_qk or norm_wide)):
+            if mix_role or unit_rms or keys_as_values:
+                raise KernelError("qkv_prep: convolutions, query multipliers and biases on values go with none of value mixing, unit_rms and keys_as_values")
+            taps, single = 0, batch.max_new_tokens == 1
+            if conv is not None:
+                taps = conv.shape[0]
+                assert conv.shape[1] == channels and (taps == 1 or tuple(conv_state.shape[1:]) == (taps - 1, channels))
+            assert q_mul is None or q_mul.numel() >= batch.max_seq_len
+            self._check(lib.llm_qkv_prep_row(
+                _ptr(parts), c_int(parts.shape[0]), c_longlong(parts.stride(0)), c_int(parts.shape[2]), c_int(heads), c_int(kv_heads), c_int(dk),
+                c_int(dv), c_int(rot_dims), _ptr(bias), c_int(0 if bias is None else bias.numel()), _ptr(conv), c_int(taps),
+                _ptr(conv_state if taps > 1 else None), c_int(1 if single else 0), _ptr(q_norm), _ptr(k_norm), c_int(1 if norm_wide else 0),
+                c_float(eps), _ptr(cos), _ptr(sin), c_int(1 if neighbours else 0), _ptr(q_mul), _ptr(batch.positions), _ptr(batch.token_seq),
+                _ptr(batch.seq_qoff), _ptr(batch.seq_slot), _ptr(block_table), c_int(block_table.shape[1]), _ptr(q_out), c_longlong(q_out.stride(0)),
+                _ptr(kcache), _ptr(vcache), c_int(page), c_int(dtype_code(q_out.dtype)), c_int(n), _stream()), lib)
+            if taps > 1 and not single:
+                self._check(lib.llm_conv_state(_ptr(parts), c_int(parts.shape[0]), c_longlong(parts.stride(0)), c_int(parts.shape[2]), c_int(0),
+                                               c_int(channels), c_int(taps), _ptr(conv_state), _ptr(batch.seq_qoff), _ptr(batch.seq_ntok),
+                                               _ptr(batch.seq_slot), c_int(batch.n_seqs), _stream()), lib)
+            return
         self._check(lib.llm_qkv_prep(_ptr(parts), c_int(parts.shape[0]), c_longlong(parts.stride(0)), c_int(parts.shape[2]), c_int(heads),
                                      c_int(kv_heads), c_int(dk), c_int(dv), c_int(rot_dims), _ptr(q_norm), _ptr(k_norm), c_float(eps),
                                      _ptr(cos), _ptr(sin), _ptr(batch.positions), _ptr(batch.token_seq), _ptr(block_table),
@@ -1204,7 +1236,7 @@ class CudaOps:
             lib = self.lib("tensorcore")
             if lib.llm_gated_attention_mma_supported(c_int(nq), c_int(nkv), c_int(dk), c_int(dv), c_longlong(q.stride(0)), c_longlong(out.stride(0))):
                 n_splits, split_keys, scratch = 1, 256, None
-                if batch.max_new_tokens == 1 and batch.n_tokens == batch.n_seqs and dk == dv:
+                if batch.max_new_tokens == 1 and batch.n_tokens == batch.n_seqs:
                     # single decoded tokens: the keys a token may see (its chunk or window at most) in pieces side by side; a
                     # window's pieces are counted from its first key's tile of 64
                     reach = min(batch.max_seq_len, chunk) if chunk > 0 else min(batch.max_seq_len, window + 63) if window > 0 else batch.max_seq_len
@@ -1383,7 +1415,8 @@ class CudaOps:
 
     def linear_state(self, rule: str, q, q_off: int, k, k_off: int, v, v_off: int, decay: torch.Tensor, decay_off: int,
                      bonus: Optional[torch.Tensor], state: torch.Tensor, batch, out: torch.Tensor, heads: int, kv_heads: int, dk: int,
-                     dv: int, q_scale: float = 1.0, unit_eps: float = -1.0, decay_const: bool = False, beta=None, beta_off: int = 0) -> torch.Tensor:
+                     dv: int, q_scale: float = 1.0, unit_eps: float = -1.0, decay_const: bool = False, beta=None, beta_off: int = 0,
+                     silu: bool = False) -> torch.Tensor:
         """Token after token of every request, per head a matrix S [dk, dv] (float32, in the request's slot of `state`):
         "decay_write_read": S <- diag(a) S + k v^T, o = S^T q; "bonus_read_decay_write": o = (S + diag(bonus) k v^T)^T q, then
         S <- diag(a) S + k v^T; "delta": S <- g S, w = beta (v - S^T k), S <- S + k w^T, o = S^T q with q and k made unit vectors
@@ -1392,7 +1425,7 @@ class CudaOps:
         ([parts, n, width] or [n, width]) read at column offsets, q and k with kv_heads heads of dk (head h reads head
         h // (heads / kv_heads)), v with heads of dv. decay: float32 rows; at decay_off a number per (head, key channel), or for
         "delta" [g: heads | beta: heads]; with decay_const a single row that holds for every token (decays that are constants
-        of the model). out float32 [n, heads * dv]."""
+        of the model); with silu, q, k and v are silu of their sums (q before its scale). out float32 [n, heads * dv]."""
         _need(decay, "linear_state.decay", torch.float32); _need(state, "linear_state.state", torch.float32); _need(out, "linear_state.out", torch.float32)
         assert decay.is_contiguous() and decay.dim() == 2 and state.is_contiguous() and out.is_contiguous() and out.shape[1] == heads * dv
         assert tuple(state.shape[1:]) == tuple(self.linear_state_shape(heads, dk, dv))
@@ -1407,7 +1440,15 @@ class CudaOps:
                                          c_int(decay.shape[1]), c_int(decay_off), _ptr(bonus), _ptr(state), _ptr(batch.seq_qoff),
                                          _ptr(batch.seq_ntok), _ptr(batch.seq_slot), _ptr(out), c_int(batch.n_tokens), c_int(batch.n_seqs), c_int(heads),
                                          c_int(kv_heads), c_int(dk), c_int(dv), c_float(q_scale), c_float(unit_eps), c_int(1 if decay_const else 0),
-                                         _stream()), lib)
+                                         c_int(1 if silu else 0), _stream()), lib)
+        return out
+
+    def silu_sums(self, x, x_off: int, columns: int, out: torch.Tensor, n_tokens: int) -> torch.Tensor:
+        """out[t] (float32 [n, columns]) = silu of `columns` columns of the float32 sums x from column x_off."""
+        _need(out, "silu_sums.out", torch.float32)
+        assert out.is_contiguous() and out.shape[1] == columns and out.shape[0] >= n_tokens
+        lib = self.lib()
+        self._check(lib.llm_silu_sums(*self._sums(x, x_off, "silu_sums.x"), c_int(columns), _ptr(out), c_int(n_tokens), _stream()), lib)
         return out
 
     def rotate_sums(self, x, x_off: int, heads: int, dk: int, cos: Optional[torch.Tensor], sin: Optional[torch.Tensor], positions: torch.Tensor,

@@ -119,17 +119,21 @@ class ParallelBlock(Block):
             else:
                 x2 = ctx.ws.get("block.norm2_out", (n, res.h.shape[1]), self.env.dtype)
                 self.norm2.run(res.h, ctx, None, n, out=x2)
+        adds = self.feed_forward is not None or self.token_input is not None  # this block adds the sums into the stream itself
+        ctx.takes_delta_bias, ctx.delta_bias = adds, None
         a = self.mixer.forward(x1, ctx, cache)
+        bias, ctx.takes_delta_bias, ctx.delta_bias = ctx.delta_bias, False, None
+        extra = {} if bias is None else {"bias": bias}
         b = self.feed_forward.forward(x2, ctx) if self.feed_forward is not None else None
         if self.token_input is None:
             if b is None:
                 res.pending = a
             else:
-                ops.stream_add(res.h, a, b, n_rows=n)
+                ops.stream_add(res.h, a, b, n_rows=n, **extra)
             res.sumsq = res.prescaled = res.prescaled_weight = res.operand = None
             return res
         xs = ctx.ws.get("block.stream_copy", (n, res.h.shape[1]), self.env.dtype)
-        ops.stream_add(res.h, a, b, copy=xs, n_rows=n)
+        ops.stream_add(res.h, a, b, copy=xs, n_rows=n, **extra)
         res.sumsq = res.prescaled = res.prescaled_weight = res.operand = None
         res.pending = self.token_input.forward(xs, ctx)
         return res

@@ -8,10 +8,12 @@ With h the mixer's input, per token at position p:
     score_a(i, j) = (q_a(i) . k_b(j)) * scale,  b = a // (H / G),  j <= i in the same chunk (and inside the window)
     p_a(i, j) = exp(score) / (sum_j exp(score) + exp(sink_a))   the sink only enlarges the denominator
     out = Wo ((heads' results side by side) * sigmoid(g))       g: a gate a number of the result, or (gate_per_head) one a head
-With q_bias and k_bias the projections of queries and keys have biases; rot_pairs "neighbours" turns the numbers 2i and 2i + 1 of a
+With q_bias, k_bias and v_bias the projections have biases, with o_bias the output projection; rot_pairs "neighbours" turns the numbers 2i and 2i + 1 of a
 head together instead of i and i + dims / 2; with unit_rms every query and key head is divided by its root mean square behind the
 rotation (no weight); with keys_as_values there is no Wv: v = k as the projection gives it, before norms and rotation.
-With norm_scope "projection" the two norms are over all of q and all of k at once (weights of the projections' sizes). A layer
+With taps > 0, q, k and v go through a causal convolution over their request's last `taps` tokens a channel, right behind the projection
+(the last taps - 1 projected rows are state); with q_temperature the queries are multiplied by a number that grows with the position;
+sink_score puts one constant in place of the sinks a head. With norm_scope "projection" the two norms are over all of q and all of k at once (weights of the projections' sizes). A layer
 without keys and values of its own (own_kv False) forms queries only and reads the cache of the run its LayerRun names.
 Norms, rotation, scores, softmax and the gate are float32 in both engine precisions. v_first are the values that the
 first layer with value mixing computed for the same tokens in the same step: that layer leaves them in the step
@@ -21,14 +23,22 @@ from __future__ import annotations
 
 from typing import List, Optional
 
+import numpy as np
 import torch
 
 from .attention import add_into_stream_or_partials
-from .base import KVNeed, LayerCache, Mixer, NormalizedRows
+from .base import KVNeed, LayerCache, Mixer, NormalizedRows, StateNeed
 from .registry import build_part, part_class, register_part
-from .spec import GatedAttentionSpec, TensorNeed
+from .spec import GatedAttentionSpec, QueryTemperatureSpec, TensorNeed
 
 V_FIRST = "gated_attention.v_first"  # key of ctx.shared
+CONV = "gated_attention.conv"        # the state's name
+
+
+def query_temperatures(spec: QueryTemperatureSpec) -> np.ndarray:
+    """What the query at every position is multiplied with, float64 rounded to float32."""
+    steps = np.floor((np.arange(spec.max_positions, dtype=np.float64) + 1.0) / float(spec.every))
+    return (1.0 + float(spec.coef) * np.log(steps + 1.0)).astype(np.float32)
 
 
 class GatedAttention(Mixer):
@@ -53,8 +63,19 @@ class GatedAttention(Mixer):
             raise ValueError("gated attention: unit_rms takes the place of the norms before the rotation")
         if spec.keys_as_values and (spec.value_dim != spec.head_dim or spec.value_mix is not None or not spec.own_kv):
             raise ValueError("gated attention: keys_as_values needs values of the keys' size, keys of the layer's own and no value mixing")
-        if (spec.q_bias or spec.k_bias or spec.unit_rms or spec.rot_pairs != "half") and spec.norm_scope != "head":
-            raise ValueError("gated attention: biases, unit_rms and neighbouring pairs go with norms a head")
+        # what the row form of the query/key/value preparation does (ops.qkv_prep): it mixes no values, has no unit_rms and no keys as values
+        self.row_form = bool(spec.taps or spec.v_bias or spec.q_temperature is not None or
+                             (spec.norm_scope == "projection" and (spec.q_bias or spec.k_bias or spec.rot_pairs != "half")))
+        if (self.row_form or spec.norm_scope == "projection") and (spec.unit_rms or spec.keys_as_values):
+            raise ValueError("gated attention: unit_rms and keys_as_values go with norms a head, without convolutions, value biases and query temperatures")
+        if self.row_form and spec.value_mix is not None:
+            raise ValueError("gated attention: convolutions, value biases and query temperatures go without value mixing")
+        if spec.taps < 0 or (spec.taps > 0 and not (spec.own_kv and spec.q_conv and spec.k_conv and spec.v_conv)):
+            raise ValueError("gated attention: a convolution needs its three weights, and keys and values of the layer's own")
+        if spec.sink and spec.sink_score is not None:
+            raise ValueError("gated attention: sinks are a tensor or one constant")
+        if spec.q_temperature is not None and not (spec.q_temperature.every > 0 and spec.q_temperature.max_positions > 0):
+            raise ValueError("gated attention: a query temperature needs a positive step and a position limit")
         self.position = build_part("position", spec.position, env)
         tables = self.position.rotation_tables()
         if tables is None:
@@ -62,7 +83,7 @@ class GatedAttention(Mixer):
         self.cos, self.sin = tables
         if self.cos is not None and 2 * self.cos.shape[1] > spec.head_dim:
             raise ValueError(f"gated attention: {2 * self.cos.shape[1]} rotated dimensions do not fit a head of {spec.head_dim}")
-        self.w_in = self.w_o = self.q_norm = self.k_norm = self.sink = self.mix = self.bias = None
+        self.w_in = self.w_o = self.q_norm = self.k_norm = self.sink = self.mix = self.bias = self.o_bias = self.conv = self.q_mul = None
 
     @staticmethod
     def tensor_needs(spec: GatedAttentionSpec) -> List[TensorNeed]:
@@ -72,9 +93,13 @@ class GatedAttention(Mixer):
             out.append(TensorNeed(spec.k_weight, (G * dk, spec.hidden)))
             if not spec.keys_as_values:
                 out.append(TensorNeed(spec.v_weight, (G * dv, spec.hidden)))
-        for name, heads in ((spec.q_bias, H), (spec.k_bias if spec.own_kv else None, G)):
+        for name, size in ((spec.q_bias, H * dk), (spec.k_bias if spec.own_kv else None, G * dk), (spec.v_bias if spec.own_kv else None, G * dv),
+                           (spec.o_bias, spec.hidden)):
             if name:
-                out.append(TensorNeed(name, (heads * dk,), "float32"))
+                out.append(TensorNeed(name, (size,), "float32"))
+        if spec.taps:
+            for name, size in ((spec.q_conv, H * dk), (spec.k_conv, G * dk), (spec.v_conv, G * dv)):
+                out.append(TensorNeed(name, (size, spec.taps), "float32"))
         if spec.gate_weight:
             out.append(TensorNeed(spec.gate_weight, (H if spec.gate_per_head else H * dv, spec.hidden)))
         wide = spec.norm_scope == "projection"
@@ -94,7 +119,14 @@ class GatedAttention(Mixer):
         s = self.spec
         if not s.own_kv:
             return ()
-        return (KVNeed(s.num_kv_heads, s.head_dim, s.window if s.cache_window is None else s.cache_window, value_dim=s.value_dim),)
+        kv = KVNeed(s.num_kv_heads, s.head_dim, s.window if s.cache_window is None else s.cache_window, value_dim=s.value_dim)
+        if s.taps > 1:
+            return (kv, StateNeed(CONV, (s.taps - 1, self._channels())))
+        return (kv,)
+
+    def _channels(self) -> int:
+        s = self.spec
+        return (s.num_heads + s.num_kv_heads) * s.head_dim + s.num_kv_heads * s.value_dim
 
     def kernel_notes(self):
         s, ops = self.spec, self.env.ops
@@ -116,11 +148,21 @@ class GatedAttention(Mixer):
         self.q_norm = tensors[s.q_norm] if s.q_norm else None
         self.k_norm = tensors[s.k_norm] if s.k_norm else None
         self.sink = tensors[s.sink] if s.sink else None
-        if s.q_bias or (s.k_bias and s.own_kv):  # one vector over the columns [q | k], zeros where a projection has none
-            zeros = lambda heads: torch.zeros(heads * s.head_dim, dtype=torch.float32, device=self.env.device)  # noqa: E731
-            q_b = tensors[s.q_bias] if s.q_bias else zeros(s.num_heads)
-            k_b = [tensors[s.k_bias] if s.k_bias else zeros(s.num_kv_heads)] if s.own_kv else []
-            self.bias = torch.cat([q_b] + k_b).contiguous()
+        if s.sink_score is not None:
+            self.sink = torch.full((s.num_heads,), float(s.sink_score), dtype=torch.float32, device=self.env.device)
+        biases = [(s.q_bias, s.num_heads * s.head_dim)]
+        if s.own_kv:
+            biases.append((s.k_bias, s.num_kv_heads * s.head_dim))
+            if s.v_bias:
+                biases.append((s.v_bias, s.num_kv_heads * s.value_dim))
+        if any(name for name, _ in biases):  # one vector over the columns [q | k] or [q | k | v], zeros where a projection has none
+            self.bias = torch.cat([tensors[name] if name else torch.zeros(size, dtype=torch.float32, device=self.env.device)
+                                   for name, size in biases]).contiguous()
+        self.o_bias = tensors[s.o_bias].contiguous() if s.o_bias else None
+        if s.taps:  # [taps, channels]: neighbouring channels read neighbouring words
+            self.conv = torch.cat([tensors[s.q_conv], tensors[s.k_conv], tensors[s.v_conv]], dim=0).t().contiguous()
+        if s.q_temperature is not None:
+            self.q_mul = torch.from_numpy(query_temperatures(s.q_temperature)).to(self.env.device)
         self.mix = tensors[s.value_mix_weight].reshape(1) if s.value_mix == "mix" else None
         self.position.load(tensors)
 
@@ -149,7 +191,10 @@ class GatedAttention(Mixer):
         q = ctx.ws.get("gated_attention.q", (n, H * dk), dt)
         writes = cache.writes and cache.k is not None and s.own_kv
         wide = {"norm_wide": True} if s.norm_scope == "projection" else {}
-        if self.bias is not None or s.unit_rms or s.rot_pairs != "half" or s.keys_as_values:
+        if self.row_form:
+            wide.update(bias=self.bias, neighbours=s.rot_pairs == "neighbours", conv=self.conv, conv_state=cache.states[CONV] if s.taps > 1 else None,
+                        q_mul=self.q_mul)
+        elif self.bias is not None or s.unit_rms or s.rot_pairs != "half" or s.keys_as_values:
             wide = {"bias": self.bias, "unit_rms": s.unit_rms, "neighbours": s.rot_pairs == "neighbours", "keys_as_values": s.keys_as_values}
         ops.qkv_prep(parts, H, G if s.own_kv else 0, dk, dv, self.q_norm, self.k_norm, s.eps, self.cos, self.sin, ctx, ctx.block_tables[cache.group], q,
                      cache.k if writes else None, cache.v if writes else None, role, self.mix, v_first, **wide)
@@ -157,7 +202,16 @@ class GatedAttention(Mixer):
         g_off = H * dk + (G * dk + (0 if s.keys_as_values else G * dv) if s.own_kv else 0)
         ops.gated_attention(q, cache.k, cache.v, ctx, ctx.block_tables[cache.group], att, H, G, dk, dv, s.scale, s.window, s.chunk,
                             self.sink, parts if s.gate_weight else None, g_off, **({"gate_per_head": True} if s.gate_per_head else {}))
-        return add_into_stream_or_partials(ops, att, self.w_o, ctx, False, "gated_attention.delta")
+        if self.o_bias is None:
+            return add_into_stream_or_partials(ops, att, self.w_o, ctx, False, "gated_attention.delta")
+        keep, ctx.residual = ctx.residual, None  # the sums are wanted here: the bias goes with them
+        delta = add_into_stream_or_partials(ops, att, self.w_o, ctx, False, "gated_attention.delta")
+        ctx.residual = keep
+        if ctx.takes_delta_bias:
+            ctx.delta_bias = self.o_bias  # the block adds it with the sums
+        else:
+            ops.stream_add(delta if delta.dim() == 2 else delta[0], None, n_rows=n, bias=self.o_bias)
+        return delta
 
 
 register_part("mixer", "gated_attention", GatedAttention)

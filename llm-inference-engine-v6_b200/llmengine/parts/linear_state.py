@@ -1,9 +1,11 @@
 """Recurrent mixers whose memory is a matrix per head, S [dk, dv] in float32, kept in the request's state slot and updated token
-after token by a rank-one write k v^T (ops.linear_state). Five of them, which differ in what decays the matrix, what is
+after token by a rank-one write k v^T (ops.linear_state). Six of them, which differ in what decays the matrix, what is
 written, and what the projections read:
 
     Retention                q, k, v, g = W h;  q and k rotated at the token's position, k times a constant;  one decay a head
                              that is a constant of the model:  S <- decay_h S + k v^T;  o = S^T q;  no weight on the heads' norm
+    LightningAttention       q, k, v = silu(W h), g = W h;  one constant decay a head as above;  S <- decay_h S + k v^T;  o = S^T q;
+                             ONE norm over all heads' results together
     DecayedLinearAttention   q, k, v, g = W h;  a = sigmoid(W_a2 (W_a1 h) + b)^(1/tau) per key channel
                              S <- diag(a) S + k v^T;  o = S^T (q dk^-1/2)
     TokenShiftMix            every projection reads its own blend h + (h_prev - h) * mu of the token's input with the previous
@@ -15,7 +17,7 @@ written, and what the projections read:
                              S <- diag(g) S;  w = beta (v - S^T k);  S <- S + k w^T;  o = S^T q
 
 All of them finish alike: every head's o divided by its root mean square, times a weight, times silu of a gate projection
-(ChannelDelta: sigmoid of a low-rank one), then the output projection. Decays, gates, unit norms, the state and o are float32 in both engine precisions; the projections'
+(ChannelDelta: sigmoid of a low-rank one; LightningAttention: sigmoid, and the norm is over all heads), then the output projection. Decays, gates, unit norms, the state and o are float32 in both engine precisions; the projections'
 float32 sums are read as they come (K-split parts are added where they are read).
 """
 from __future__ import annotations
@@ -27,7 +29,13 @@ import torch
 from .attention import add_into_stream_or_partials, project_sums
 from .base import LayerCache, Mixer, NormalizedRows, StateNeed
 from .registry import build_part, part_class, register_part
-from .spec import ChannelDeltaSpec, DecayedLinearAttentionSpec, GatedDeltaSpec, RetentionSpec, TensorNeed, TokenShiftMixSpec
+from .spec import ChannelDeltaSpec, DecayedLinearAttentionSpec, GatedDeltaSpec, LightningAttentionSpec, RetentionSpec, TensorNeed, TokenShiftMixSpec
+
+
+def _constant_decays(decay, dim: int, device) -> torch.Tensor:
+    """One decay a head as linear_state reads constants: a number a (head, key channel), one row for all tokens; float32 from the
+    configuration's doubles."""
+    return torch.tensor(decay, dtype=torch.float64).to(torch.float32).repeat_interleave(dim).reshape(1, len(decay) * dim).contiguous().to(device)
 
 
 def _state_shape(env, heads: int, dk: int, dv: int):
@@ -114,8 +122,7 @@ class Retention(Mixer):
         s, dev = self.spec, self.env.device
         self.w_in = torch.cat([tensors[s.q_weight], tensors[s.k_weight], tensors[s.v_weight], tensors[s.g_weight]], dim=0).contiguous()
         self.w_o = tensors[s.o_weight]
-        # the decays as the kernel reads them: a number a (head, key channel), one row for all tokens; float32 from the configuration's doubles
-        self.decay = torch.tensor(s.decay, dtype=torch.float64).to(torch.float32).repeat_interleave(s.dim).reshape(1, s.heads * s.dim).contiguous().to(dev)
+        self.decay = _constant_decays(s.decay, s.dim, dev)
         self.ones = torch.ones(s.vdim, dtype=torch.float32, device=dev)
         self.position.load(tensors)
 
@@ -133,6 +140,55 @@ class Retention(Mixer):
         y = ctx.ws.get("retention.y", (n, H * dv), dt)
         ops.head_norm_gate(o, self.ones, sums, 2 * H * dk + H * dv, s.eps, y, n, H, dv)
         return add_into_stream_or_partials(ops, y, self.w_o, ctx, False, "retention.delta")
+
+
+class LightningAttention(Mixer):
+    """Linear attention with a fixed decay per head over activated projections (LightningAttentionSpec). The state walks the tokens under
+    the rule "decay_write_read" with one constant row of decays. silu of q, k and v: in a step of few tokens the kernel applies it where
+    it adds the projections' parts; a portion's sums are activated by a kernel of their own, since every block of a head would do it
+    again. The norm over all heads' results is head_norm_gate with the heads as one."""
+
+    ACTIVATE_APART_FROM = 65  # tokens of a step
+
+    def __init__(self, spec: LightningAttentionSpec, env):
+        super().__init__(spec, env)
+        if min(spec.heads, spec.dim, spec.vdim) <= 0 or len(spec.decay) != spec.heads:
+            raise ValueError("lightning attention: sizes must be positive, and there is one decay a head")
+        self.w_in = self.w_o = self.decay = self.norm_w = None
+
+    @staticmethod
+    def tensor_needs(spec: LightningAttentionSpec) -> List[TensorNeed]:
+        H, dk, dv, D = spec.heads, spec.dim, spec.vdim, spec.hidden
+        return [TensorNeed(spec.q_weight, (H * dk, D)), TensorNeed(spec.k_weight, (H * dk, D)), TensorNeed(spec.v_weight, (H * dv, D)),
+                TensorNeed(spec.g_weight, (H * dv, D)), TensorNeed(spec.norm_weight, (H * dv,), "float32", init="around_one"),
+                TensorNeed(spec.o_weight, (D, H * dv))]
+
+    def cache_needs(self):
+        s = self.spec
+        return (StateNeed("lightning.state", _state_shape(self.env, s.heads, s.dim, s.vdim)),)
+
+    def load(self, tensors) -> None:
+        s = self.spec
+        self.w_in = torch.cat([tensors[s.q_weight], tensors[s.k_weight], tensors[s.v_weight], tensors[s.g_weight]], dim=0).contiguous()
+        self.w_o, self.norm_w = tensors[s.o_weight], tensors[s.norm_weight].contiguous()
+        self.decay = _constant_decays(s.decay, s.dim, self.env.device)
+
+    def forward(self, x, ctx, cache: LayerCache) -> Optional[torch.Tensor]:
+        s, ops, n, dt = self.spec, self.env.ops, ctx.n_tokens, self.env.dtype
+        if isinstance(x, NormalizedRows):
+            x = x.dense(ctx)
+        H, dk, dv = s.heads, s.dim, s.vdim
+        qkv = 2 * H * dk + H * dv
+        sums = project_sums(ops, ctx, x, self.w_in, "lightning.in")  # [q | k | v | g], float32, never rounded
+        acts, inside = sums, True
+        if n >= self.ACTIVATE_APART_FROM:
+            acts, inside = ops.silu_sums(sums, 0, qkv, ctx.ws.get("lightning.qkv", (n, qkv), torch.float32), n), False
+        o = ctx.ws.get("lightning.o", (n, H * dv), torch.float32)
+        ops.linear_state("decay_write_read", acts, 0, acts, H * dk, acts, 2 * H * dk, self.decay, 0, None, cache.states["lightning.state"], ctx, o,
+                         H, H, dk, dv, decay_const=True, silu=inside)
+        y = ctx.ws.get("lightning.y", (n, H * dv), dt)
+        ops.head_norm_gate(o, self.norm_w, sums, qkv, s.eps, y, n, 1, H * dv, act="sigmoid")
+        return add_into_stream_or_partials(ops, y, self.w_o, ctx, False, "lightning.delta")
 
 
 class TokenShiftMix(Mixer):
@@ -296,6 +352,7 @@ class ChannelDelta(Mixer):
 
 
 register_part("mixer", "retention", Retention)
+register_part("mixer", "lightning_attention", LightningAttention)
 register_part("mixer", "decayed_linear_attention", DecayedLinearAttention)
 register_part("mixer", "token_shift_mix", TokenShiftMix)
 register_part("mixer", "gated_delta", GatedDelta)

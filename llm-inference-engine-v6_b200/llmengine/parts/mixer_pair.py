@@ -53,11 +53,11 @@ class MixerPair(Mixer):
         s, ops, n = self.spec, self.env.ops, ctx.n_tokens
         if isinstance(x, NormalizedRows):
             x = x.dense(ctx)
-        keep = ctx.residual
-        ctx.residual = None  # neither side adds into the stream: their sums are put together first
+        keep, keep_bias = ctx.residual, ctx.takes_delta_bias
+        ctx.residual, ctx.takes_delta_bias = None, False  # neither side adds into the stream: their whole sums are put together first
         a = self.left.forward(x, ctx, cache)
         b = self.right.forward(x, ctx, cache)
-        ctx.residual = keep
+        ctx.residual, ctx.takes_delta_bias = keep, keep_bias
         out = ctx.ws.get("mixer_pair.delta", (n, s.hidden), torch.float32)
         if s.combine == "weighted":
             return ops.pair_combine(a, b, None, None, s.left_scale, s.right_scale, 0.0, out, n)

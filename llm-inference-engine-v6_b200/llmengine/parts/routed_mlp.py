@@ -73,7 +73,7 @@ class RoutedMLP(FeedForward):
 
 
 class GroupRoutedMLP(FeedForward):
-    """Gated experts chosen by scores over all experts, with a correction that only the choice sees and a limit on groups
+    """Gated experts (or, without gate matrices, experts of two matrices around one activation) chosen by scores over all experts, with a correction that only the choice sees and a limit on groups
     of experts (GroupRoutedMLPSpec), plus an optional expert that every token goes through:
 
         s = softmax(Wr x) or sigmoid(Wr x)  (float32);  choice = s + correction;  only the best `keep_groups` of `groups` groups stay
@@ -85,6 +85,10 @@ class GroupRoutedMLP(FeedForward):
     `identity` > 0 the router has that many more outputs behind the experts' whose "expert" returns x itself: they take part in
     scores and choice like the others, get no tiles in the per-expert products, and are added where the chosen rows are summed.
 
+    Experts without gate matrices: Wdown_e act(Wup_e x), act the square of relu. With weigh "input" the weight multiplies what an expert
+    reads, sum_e Wdown_e act(Wup_e (g_e x)): the first matrix is linear, so its product's epilogue applies act(g_e * sum) and the
+    second product carries no weight.
+
     An expert's gate and up rows are stored in turn ([E, 2 ff, hidden]: row 2 f the gate, row 2 f + 1 its up row), so that the
     per-expert product has both in one thread's hands and applies silu(gate) * up in its epilogue. Where the caller says that
     it takes pairs (ctx.takes_delta_pairs: a block that adds two sets of sums in one kernel), the routed sum and the shared
@@ -92,8 +96,13 @@ class GroupRoutedMLP(FeedForward):
 
     def __init__(self, spec: GroupRoutedMLPSpec, env):
         super().__init__(spec, env)
-        if spec.activation not in ("silu", "clamped_swish") or (spec.activation == "clamped_swish" and not spec.limit > 0):
+        self.gated = len(spec.gate_weights) > 0
+        if self.gated and (spec.activation not in ("silu", "clamped_swish") or (spec.activation == "clamped_swish" and not spec.limit > 0)):
             raise ValueError(f"routed gated feed-forward: activation '{spec.activation}' is not implemented (silu and clamped_swish with a positive limit are)")
+        if not self.gated and spec.activation != "relu_squared":
+            raise ValueError(f"routed feed-forward without gates: activation '{spec.activation}' is not implemented (relu_squared is)")
+        if spec.weigh not in ("input", "output") or (spec.weigh == "input" and (self.gated or spec.identity)):
+            raise ValueError("routed feed-forward: weigh is 'output', or for experts without gates and without identity experts 'input'")
         self.act = (spec.activation, float(spec.limit), float(spec.slope)) if spec.activation == "clamped_swish" else spec.activation
         if spec.identity < 0 or (spec.shared_gate and spec.shared is None):
             raise ValueError("routed feed-forward: identity experts cannot be negative, and a gate on the shared expert needs one")
@@ -106,10 +115,10 @@ class GroupRoutedMLP(FeedForward):
             raise ValueError("routed feed-forward: score is 'softmax' or 'sigmoid', a group's score sums its 1 or 2 largest")
         if spec.keep_groups * (self.outputs // spec.groups) < spec.top:
             raise ValueError("routed feed-forward: the groups that stay hold fewer experts than a token uses")
-        if not (len(spec.gate_weights) == len(spec.up_weights) == len(spec.down_weights) == spec.experts):
-            raise ValueError("routed feed-forward: one gate, one up and one down matrix per expert")
+        if not (len(spec.up_weights) == len(spec.down_weights) == spec.experts and len(spec.gate_weights) in (0, spec.experts)):
+            raise ValueError("routed feed-forward: one up and one down matrix per expert, and a gate matrix for all of them or none")
         self.shared = build_part("feed_forward", spec.shared, env) if spec.shared is not None else None
-        self.router = self.correction = self.w_gate_up = self.w_down = None
+        self.router = self.correction = self.w_up = self.w_down = None
 
     @staticmethod
     def tensor_needs(spec: GroupRoutedMLPSpec) -> List[TensorNeed]:
@@ -119,9 +128,10 @@ class GroupRoutedMLP(FeedForward):
             out.append(TensorNeed(spec.correction, (outputs,), "float32", init="zeros"))
         if spec.shared_gate:
             out.append(TensorNeed(spec.shared_gate, (1, spec.hidden)))
-        for g, u, d in zip(spec.gate_weights, spec.up_weights, spec.down_weights):
-            out += [TensorNeed(g, (spec.intermediate, spec.hidden)), TensorNeed(u, (spec.intermediate, spec.hidden)),
-                    TensorNeed(d, (spec.hidden, spec.intermediate))]
+        for g in spec.gate_weights:
+            out.append(TensorNeed(g, (spec.intermediate, spec.hidden)))
+        for u, d in zip(spec.up_weights, spec.down_weights):
+            out += [TensorNeed(u, (spec.intermediate, spec.hidden)), TensorNeed(d, (spec.hidden, spec.intermediate))]
         if spec.shared is not None:
             out += part_class("feed_forward", spec.shared.kind).tensor_needs(spec.shared)
         return out
@@ -142,8 +152,11 @@ class GroupRoutedMLP(FeedForward):
         if s.shared_gate:  # the shared expert's gate is one more row behind the router's: the routing kernel forms both in float32
             self.router = torch.cat([self.router, tensors[s.shared_gate].reshape(1, s.hidden)], dim=0).contiguous()
         self.correction = tensors[s.correction] if s.correction else None
-        gu = [torch.stack([tensors[g], tensors[u]], dim=1).reshape(2 * s.intermediate, s.hidden) for g, u in zip(s.gate_weights, s.up_weights)]
-        self.w_gate_up = torch.stack(gu).contiguous()                                  # [E, 2 ff, hidden], gate and up rows in turn
+        if self.gated:
+            gu = [torch.stack([tensors[g], tensors[u]], dim=1).reshape(2 * s.intermediate, s.hidden) for g, u in zip(s.gate_weights, s.up_weights)]
+            self.w_up = torch.stack(gu).contiguous()                                   # [E, 2 ff, hidden], gate and up rows in turn
+        else:
+            self.w_up = torch.stack([tensors[n] for n in s.up_weights]).contiguous()  # [E, ff, hidden]
         self.w_down = torch.stack([tensors[n] for n in s.down_weights]).contiguous()  # [E, hidden, ff]
         if self.shared is not None:
             self.shared.load(tensors)
@@ -170,12 +183,17 @@ class GroupRoutedMLP(FeedForward):
         else:
             tile_expert, tile_rows = ops.routed_group(idx, s.experts, tile, ctx.ws, "routed")
         act = ctx.ws.get("routed.act", (n * s.top, s.intermediate), dt)
-        if s.activation == "silu":
-            ops.routed_product(x, s.top, self.w_gate_up, tile_expert, tile_rows, act, "silu_pairs")
+        on_input, on_output = (share.view(-1), None) if s.weigh == "input" else (None, share.view(-1))
+        if not self.gated:
+            ops.routed_product(x, s.top, self.w_up, tile_expert, tile_rows, act, "relu_squared", share=on_input)
+        elif s.activation == "silu":
+            ops.routed_product(x, s.top, self.w_up, tile_expert, tile_rows, act, "silu_pairs")
         else:
-            ops.routed_product(x, s.top, self.w_gate_up, tile_expert, tile_rows, act, "gated_pairs", act=self.act)
+            ops.routed_product(x, s.top, self.w_up, tile_expert, tile_rows, act, "gated_pairs", act=self.act)
         y = ctx.ws.get("routed.y", (n * s.top, s.hidden), torch.float32)
-        ops.routed_product(act, 1, self.w_down, tile_expert, tile_rows, y, "share", share=share.view(-1))
+        ops.routed_product(act, 1, self.w_down, tile_expert, tile_rows, y, "share", share=on_output)
+        if s.top == 1 and not s.identity and self.shared is None:
+            return y  # one expert a token: its row, written at the token's own index, is the sum
         identity = (idx, share, s.experts, x) if s.identity else None
         out = ctx.ws.get("routed.delta", (n, s.hidden), torch.float32)
         if self.shared is None:

@@ -131,6 +131,15 @@ class AttentionSpec:
 
 
 @dataclass(frozen=True)
+class QueryTemperatureSpec:
+    """What a query at position p is multiplied with: 1 + coef * ln(floor((p + 1) / every) + 1), in float32 (a table of max_positions
+    numbers made from float64 ones)."""
+    coef: float
+    every: float
+    max_positions: int
+
+
+@dataclass(frozen=True)
 class GatedAttentionSpec:
     """Causal grouped-query attention with keys of `head_dim` and values of `value_dim` numbers a head (kind "gated_attention",
     parts/gated_attention.py). Options, each off when its field is None / 0 / False:
@@ -146,10 +155,14 @@ class GatedAttentionSpec:
     own_kv False: the layer has no key and value projections (no k_weight, v_weight, k_norm): its run reads the cache of the run that
     LayerRun.cache_from names, keys as that layer normalised and rotated them. cache_window: how many of the last keys the cache
     must keep when that is more than this layer's own window asks for, because borrowers look further back (None: `window`; 0: all).
-    q_bias, k_bias: vectors added to the projections of queries and keys. rot_pairs: which numbers of a head turn together, "half"
+    q_bias, k_bias, v_bias, o_bias: vectors added to the projections of queries, keys and values and to the output projection. rot_pairs: which numbers of a head turn together, "half"
     (i with i + dims / 2) or "neighbours" (2i with 2i + 1). unit_rms: every query and key head is divided by its root mean square
     over head_dim (eps inside the root, no weight) AFTER the rotation. keys_as_values: there is no value projection, a head's values
-    are its keys as the projection (with its bias) gives them, before any norm and rotation (value_dim == head_dim)."""
+    are its keys as the projection (with its bias) gives them, before any norm and rotation (value_dim == head_dim).
+    sink_score: a sink with this score in every head in place of a tensor's (0: one is added to the softmax's denominator).
+    q_temperature: the queries are multiplied by a number that their position gives. taps > 0: q, k and v each go through a causal
+    convolution of `taps` inputs a channel (q_conv, k_conv, v_conv [channels, taps], no bias, no activation) right behind the
+    projection, before norms and rotation; the last taps - 1 projected rows of a request are its state."""
     kind: str
     hidden: int
     num_heads: int
@@ -180,6 +193,14 @@ class GatedAttentionSpec:
     rot_pairs: str = "half"                # "half" | "neighbours"
     unit_rms: bool = False
     keys_as_values: bool = False
+    v_bias: Optional[str] = None
+    o_bias: Optional[str] = None
+    sink_score: Optional[float] = None
+    q_temperature: Optional[QueryTemperatureSpec] = None
+    taps: int = 0
+    q_conv: Optional[str] = None
+    k_conv: Optional[str] = None
+    v_conv: Optional[str] = None
 
 
 @dataclass(frozen=True)
@@ -249,6 +270,26 @@ class RetentionSpec:
     k_weight: str
     v_weight: str
     g_weight: str
+    o_weight: str
+
+
+@dataclass(frozen=True)
+class LightningAttentionSpec:
+    """Linear attention with one fixed decay per head over activated projections (kind "lightning_attention", parts/linear_state.py):
+    q = silu(Wq h), k = silu(Wk h) (heads x dim), v = silu(Wv h) (heads x vdim); S <- decay_h S + k v^T; o = S^T q; ALL heads' o side by
+    side are divided by their common root mean square (eps) and multiplied by norm_weight [heads * vdim]; out = Wo (o * sigmoid(Wg h))."""
+    kind: str
+    hidden: int
+    heads: int
+    dim: int
+    vdim: int
+    decay: Tuple[float, ...]
+    eps: float
+    q_weight: str
+    k_weight: str
+    v_weight: str
+    g_weight: str
+    norm_weight: str
     o_weight: str
 
 
@@ -403,7 +444,9 @@ class GroupRoutedMLPSpec:
     and `slope` as in GatedMLPSpec); `shared` (a GatedMLPSpec or None) runs for every token and is added, times
     sigmoid(shared_gate . x) (a tensor [1, hidden]) if shared_gate names one. identity: the router has `experts + identity`
     outputs, and the last `identity` of them are experts without tensors whose result is the input x itself (scores, correction,
-    groups and the choice run over all experts + identity outputs)."""
+    groups and the choice run over all experts + identity outputs). No gate_weights: an expert is down_e(act(up_e x)) (activation
+    "relu_squared": the square of max(z, 0)). weigh "input": a chosen expert's weight multiplies what the expert reads instead of what
+    it gives: sum of expert_e(g_e x) (experts without gate matrices, no identity experts)."""
     kind: str
     hidden: int
     intermediate: int
@@ -427,6 +470,7 @@ class GroupRoutedMLPSpec:
     shared_gate: Optional[str] = None
     limit: float = 0.0
     slope: float = 1.0
+    weigh: str = "output"
 
 
 @dataclass(frozen=True)

@@ -112,8 +112,10 @@ class CpuOps:
         return self.silu_mul(gate_up, out, 128, act)
 
     # ------------------------------------------------------------------ stream, token side input
-    def stream_add(self, h, a, b=None, copy=None, n_rows=None):
+    def stream_add(self, h, a, b=None, copy=None, n_rows=None, bias=None):
         n = h.shape[0] if n_rows is None else n_rows
+        if bias is not None:
+            h[:n] += bias
         for d in (a, b):
             if d is not None:
                 h[:n] += (d if d.dim() == 2 else d.sum(0))[:n]
@@ -252,7 +254,9 @@ class CpuOps:
                 if epilogue == "gelu":
                     v = 0.5 * v * (1.0 + torch.erf(v / 2.0 ** 0.5))
                 elif epilogue == "share":
-                    v = v * share[p]
+                    v = v if share is None else v * share[p]
+                elif epilogue == "relu_squared":
+                    v = torch.clamp(v if share is None else v * share[p], min=0) ** 2
                 elif epilogue == "gated_pairs":
                     v = self._glu(v[0::2], v[1::2], act)
                 else:  # "silu_pairs": rows 2 f and 2 f + 1 are a gate and its up row
@@ -313,8 +317,19 @@ class CpuOps:
 
     def qkv_prep(self, parts, heads, kv_heads, dk, dv, q_norm, k_norm, eps, cos, sin, batch, block_table, q_out, kcache, vcache,
                  mix_role=0, mix_weight=None, v_first=None, norm_wide=False, bias=None, neighbours=False, unit_rms=False,
-                 keys_as_values=False):
+                 keys_as_values=False, conv=None, conv_state=None, q_mul=None):
         src = parts.sum(0)
+        if conv is not None:
+            src = src.clone()
+            K, C = conv.shape
+            for s in range(batch.n_seqs):
+                first, n, slot = int(batch.seq_qoff[s]), int(batch.seq_ntok[s]), int(batch.seq_slot[s])
+                x = src[first:first + n, :C].clone()
+                padded = torch.cat([conv_state[slot], x], dim=0) if K > 1 else x
+                for t in range(n):
+                    src[first + t, :C] = (conv * padded[t:t + K]).sum(0)
+                if K > 1:
+                    conv_state[slot] = padded[padded.shape[0] - (K - 1):]
         if bias is not None:
             src = src.clone()
             src[:, :bias.numel()] += bias
@@ -338,6 +353,8 @@ class CpuOps:
                     x[:, ib] = b * cos[pos] + a * sin[pos]
                 if unit_rms and x.numel():
                     x.copy_(x / torch.sqrt((x * x).mean(-1, keepdim=True) + eps))
+            if q_mul is not None:
+                q = q * q_mul[pos]
             if mix_role == 1:
                 v_first[t] = v
             elif mix_role == 2:
@@ -447,10 +464,11 @@ class CpuOps:
         return (t if t.dim() == 2 else t.sum(0))[:, off:off + width]
 
     def linear_state(self, rule, q, q_off, k, k_off, v, v_off, decay, decay_off, bonus, state, batch, out, heads, kv_heads, dk, dv,
-                     q_scale=1.0, unit_eps=-1.0, decay_const=False, beta=None, beta_off=0):
-        Q = self._cols(q, q_off, kv_heads * dk).reshape(-1, kv_heads, dk) * q_scale
-        K = self._cols(k, k_off, kv_heads * dk).reshape(-1, kv_heads, dk)
-        V = self._cols(v, v_off, heads * dv).reshape(-1, heads, dv)
+                     q_scale=1.0, unit_eps=-1.0, decay_const=False, beta=None, beta_off=0, silu=False):
+        act = torch.nn.functional.silu if silu else (lambda t: t)
+        Q = act(self._cols(q, q_off, kv_heads * dk)).reshape(-1, kv_heads, dk) * q_scale
+        K = act(self._cols(k, k_off, kv_heads * dk)).reshape(-1, kv_heads, dk)
+        V = act(self._cols(v, v_off, heads * dv)).reshape(-1, heads, dv)
         strength = self._cols(beta, beta_off, heads) if beta is not None else None
         if rule in ("delta", "channel_delta") and unit_eps >= 0:
             Q = Q / torch.sqrt((Q / q_scale).pow(2).sum(-1, keepdim=True) + unit_eps)
@@ -483,6 +501,10 @@ class CpuOps:
                         S = a[:, :, None] * S + kv
                 out[t] = o.reshape(-1)
             state[slot] = S
+        return out
+
+    def silu_sums(self, x, x_off, columns, out, n_tokens):
+        out[:n_tokens] = torch.nn.functional.silu(self._cols(x, x_off, columns)[:n_tokens])
         return out
 
     def rotate_sums(self, x, x_off, heads, dk, cos, sin, positions, out, n_tokens, scaled_from=None, scale=1.0):
