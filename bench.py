@@ -559,7 +559,40 @@ ZUDATAR_SIZES = {
     "w1024": (zudatar_sizes(1024, 16, 4, 64, 1024, 8, 64, 256, 384, 8, 128, 64, 2816, 4, 32768), sogutar_dense(SOGUTAR_SIZES["w1024"][0])),
     "w2048": (zudatar_sizes(2048, 32, 8, 64, 1024, 16, 128, 512, 768, 16, 128, 128, 8192, 4, 32768), sogutar_dense(SOGUTAR_SIZES["w2048"][0])),
 }
-DESIGNS = {"vapelix": DESIGN_SIZES, "zulopel": ZULOPEL_SIZES, "selinex": SELINEX_SIZES, "sogutar": SOGUTAR_SIZES, "zudatar": ZUDATAR_SIZES}
+
+
+def kasarax_sizes(width, heads, kv_heads, dim, state_heads, state_dim, ff, experts, top, expert_ff, layers, vocab):
+    a = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5}
+    left = dict(a, conv=4, rot={"dims": dim // 2, "base": 500000.0})
+    right = {"heads": state_heads, "dim": state_dim // 2, "vdim": state_dim, "decay": [1.0 - 2.0 ** (-1.0 - 9.0 * h / max(state_heads - 1, 1)) for h in range(state_heads)]}
+    pair = {"left": left, "right": right}
+    att = dict(a, vdim=dim // 2, q_temp={"coef": 0.1, "every": 1024})
+    dense = {"kind": "dense", "ff": ff}
+    moe = {"kind": "moe", "expert": {"ff": expert_ff}, "router": {"experts": experts, "top": top}}
+    kinds = [("parallel", pair, dense), ("parallel", pair, moe), ("attention", att, moe), ("parallel", pair, dense)]
+    return {"architecture": "Kasarax", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "logit_scale": 0.25, "max_positions": 8192,
+            "layers": [{"type": t, "mixer": m, "mlp": f} for t, m, f in (kinds[i % 4] for i in range(layers))]}
+
+
+def selinex_pairs(cfg):
+    """The Selinex configuration with pairs of mixers in three of four layers, attention without windows, and dense and routed
+    feed-forwards in the same places as the Kasarax configuration."""
+    pair, delta = next(l["mixer"] for l in cfg["layers"] if l["type"] == "parallel"), next(l["mixer"] for l in cfg["layers"] if l["type"] == "delta")
+    dense, moe = (next(l["mlp"] for l in cfg["layers"] if l["mlp"]["kind"] == k) for k in ("dense", "moe"))
+    pair = dict(pair, left={k: v for k, v in pair["left"].items() if k != "mask"})
+    kinds = [("parallel", pair, dense), ("parallel", pair, moe), ("delta", delta, moe), ("parallel", pair, dense)]
+    return dict(cfg, layers=[{"type": t, "mixer": m, "mlp": f} for t, m, f in (kinds[i % 4] for i in range(len(cfg["layers"])))])
+
+
+# Kasarax: attention behind short convolutions beside lightning attention in three of four layers, attention with biases and a query
+# temperature in the other, dense feed-forwards and experts of two matrices (of 3/2 the inner size, so that an expert weighs as much
+# as a gated one); beside it a Selinex configuration (attention beside a linear state in three of four layers, routed experts by
+# sigmoid scores: the closest existing model) of the same sizes
+KASARAX_SIZES = {
+    "w1024": (kasarax_sizes(1024, 16, 4, 64, 8, 128, 2816, 8, 2, 2112, 4, 32768), selinex_pairs(SELINEX_SIZES["w1024"][0])),
+    "w2048": (kasarax_sizes(2048, 32, 8, 64, 16, 128, 8192, 16, 4, 3072, 4, 32768), selinex_pairs(SELINEX_SIZES["w2048"][0])),
+}
+DESIGNS = {"kasarax": KASARAX_SIZES, "vapelix": DESIGN_SIZES, "zulopel": ZULOPEL_SIZES, "selinex": SELINEX_SIZES, "sogutar": SOGUTAR_SIZES, "zudatar": ZUDATAR_SIZES}
 
 
 def run_design(args):

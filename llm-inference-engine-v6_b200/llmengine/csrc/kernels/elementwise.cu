@@ -508,10 +508,52 @@ __global__ void stream_add_kernel(float* __restrict__ h, const float* __restrict
   if (copy) copy[i] = from_f32<T>(x);
 }
 
+// The same for totals and rows of a multiple of 4 numbers behind 16-byte aligned pointers: a thread moves four neighbouring numbers.
+template <typename T>
+__global__ void __launch_bounds__(256)
+    stream_add_vec_kernel(float* __restrict__ h, const float* __restrict__ a, int na, size_t sa, const float* __restrict__ b, int nb, size_t sb,
+                          T* __restrict__ copy, size_t total, const float* __restrict__ bias, int dim) {
+  dep_launch();
+  dep_wait();
+  const size_t i = ((size_t)blockIdx.x * blockDim.x + threadIdx.x) * 4;
+  if (i >= total) return;
+  float4 x = *reinterpret_cast<const float4*>(h + i);
+  auto add = [&](const float* p, int n, size_t stride) {
+    float4 d = *reinterpret_cast<const float4*>(p + i);
+#pragma unroll 4
+    for (int k = 1; k < n; ++k) {
+      const float4 v = *reinterpret_cast<const float4*>(p + (size_t)k * stride + i);
+      d.x += v.x; d.y += v.y; d.z += v.z; d.w += v.w;
+    }
+    x.x += d.x; x.y += d.y; x.z += d.z; x.w += d.w;
+  };
+  if (a) add(a, na, sa);
+  if (bias) {
+    const float4 v = *reinterpret_cast<const float4*>(bias + i % dim);
+    x.x += v.x; x.y += v.y; x.z += v.z; x.w += v.w;
+  }
+  if (b) add(b, nb, sb);
+  *reinterpret_cast<float4*>(h + i) = x;
+  if (copy) store4<T>(copy + i, x.x, x.y, x.z, x.w);
+}
+
 extern "C" int llm_stream_add(float* h, const float* a, int na, long long sa, const float* b, int nb, long long sb, void* copy,
                               int copy_dtype, long long total, const float* bias, int dim, cudaStream_t stream) {
   if (total == 0) return LLM_OK;
   LLM_REQUIRE(bias == nullptr || dim > 0, "stream_add: a bias needs the row's size");
+  LLM_REQUIRE(copy_dtype == LLM_F32 || copy_dtype == LLM_BF16, "stream_add: unknown dtype %d", copy_dtype);
+  auto al16 = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15u) == 0; };
+  if (total > 0 && total % 4 == 0 && (bias == nullptr || dim % 4 == 0) && sa % 4 == 0 && sb % 4 == 0 && al16(h) && al16(a) && al16(b) && al16(copy) && al16(bias) &&
+      (a == nullptr || na >= 1) && (b == nullptr || nb >= 1)) {
+    // few tokens: small blocks, so that the parts are read by many multiprocessors side by side
+    const int threads = total <= 148 * 1024 ? 64 : 256, vblocks = ceil_div(total / 4, threads);
+    if (copy_dtype == LLM_F32)
+      launch_kernel(stream_add_vec_kernel<float>, vblocks, threads, 0, stream, h, a, na, (size_t)sa, b, nb, (size_t)sb, (float*)copy, (size_t)total, bias, dim);
+    else
+      launch_kernel(stream_add_vec_kernel<bf16>, vblocks, threads, 0, stream, h, a, na, (size_t)sa, b, nb, (size_t)sb, (bf16*)copy, (size_t)total, bias, dim);
+    LLM_CHECK_LAUNCH("stream_add");
+    return LLM_OK;
+  }
   LLM_REQUIRE(total > 0 && (a == nullptr || na >= 1) && (b == nullptr || nb >= 1), "stream_add: bad sizes");
   const int blocks = ceil_div(total, 256);
   if (copy_dtype == LLM_F32)
@@ -743,12 +785,69 @@ __global__ void __launch_bounds__(256)
     out[base + i] = ca * ya + cb * yb;
   }
 }
+
+// The same for rows of a multiple of 4 numbers behind 16-byte aligned pointers: a thread has up to PC_GROUPS groups of four neighbouring
+// numbers of both rows, every part is read once, four parts of both sets of sums in flight, and the sums stay in registers between the
+// statistic and the result.
+constexpr int PC_GROUPS = 2;
+__device__ __forceinline__ void add4(float4& x, const float4& v) { x.x += v.x; x.y += v.y; x.z += v.z; x.w += v.w; }
+__device__ __forceinline__ float squares4(const float4& x) { return x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w; }
+__global__ void __launch_bounds__(1024)
+    pair_combine_vec_kernel(const float* __restrict__ a, int na, size_t sa, const float* __restrict__ b, int nb, size_t sb,
+                            const float* __restrict__ wa, const float* __restrict__ wb, float ca, float cb, float eps, float* __restrict__ out, int dim) {
+  __shared__ float red[33];
+  dep_launch();
+  dep_wait();
+  const size_t base = (size_t)blockIdx.x * dim;
+  const int both = min(na, nb);
+  float4 ya[PC_GROUPS], yb[PC_GROUPS];
+  float ssa = 0.f, ssb = 0.f;
+#pragma unroll
+  for (int k = 0; k < PC_GROUPS; ++k) {
+    const int i = 4 * (threadIdx.x + k * blockDim.x);
+    ya[k] = yb[k] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (i >= dim) continue;
+    const float* pa = a + base + i;
+    const float* pb = b + base + i;
+    ya[k] = *reinterpret_cast<const float4*>(pa);
+    yb[k] = *reinterpret_cast<const float4*>(pb);
+#pragma unroll 4
+    for (int p = 1; p < both; ++p) {
+      add4(ya[k], *reinterpret_cast<const float4*>(pa + (size_t)p * sa));
+      add4(yb[k], *reinterpret_cast<const float4*>(pb + (size_t)p * sb));
+    }
+#pragma unroll 4
+    for (int p = both; p < na; ++p) add4(ya[k], *reinterpret_cast<const float4*>(pa + (size_t)p * sa));
+#pragma unroll 4
+    for (int p = both; p < nb; ++p) add4(yb[k], *reinterpret_cast<const float4*>(pb + (size_t)p * sb));
+    ssa += squares4(ya[k]);
+    ssb += squares4(yb[k]);
+  }
+  const float inv_a = wa ? ca / sqrtf(block_sum(ssa, red) / (float)dim + eps) : ca;
+  const float inv_b = wb ? cb / sqrtf(block_sum(ssb, red) / (float)dim + eps) : cb;
+  const float4 ones = make_float4(1.f, 1.f, 1.f, 1.f);
+#pragma unroll
+  for (int k = 0; k < PC_GROUPS; ++k) {
+    const int i = 4 * (threadIdx.x + k * blockDim.x);
+    if (i >= dim) continue;
+    const float4 u = wa ? *reinterpret_cast<const float4*>(wa + i) : ones, v = wb ? *reinterpret_cast<const float4*>(wb + i) : ones;
+    *reinterpret_cast<float4*>(out + base + i) = make_float4(ya[k].x * inv_a * u.x + yb[k].x * inv_b * v.x, ya[k].y * inv_a * u.y + yb[k].y * inv_b * v.y,
+                                                              ya[k].z * inv_a * u.z + yb[k].z * inv_b * v.z, ya[k].w * inv_a * u.w + yb[k].w * inv_b * v.w);
+  }
+}
 }  // namespace
 
 extern "C" int llm_pair_combine(const float* a, int na, long long sa, const float* b, int nb, long long sb, const float* wa, const float* wb,
                                 float ca, float cb, float eps, float* out, int n_rows, int dim, cudaStream_t stream) {
   if (n_rows == 0) return LLM_OK;
   LLM_REQUIRE(n_rows > 0 && dim > 0 && a && b && na >= 1 && nb >= 1 && out, "pair_combine: bad arguments");
+  auto al16 = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15u) == 0; };
+  if (dim % 4 == 0 && dim <= 4 * 1024 * PC_GROUPS && al16(a) && al16(b) && al16(wa) && al16(wb) && al16(out) && sa % 4 == 0 && sb % 4 == 0) {
+    const int threads = min(1024, ceil_div(dim, 128) * 32);  // the row's size alone decides, and with it the order of the sums of squares
+    launch_kernel(pair_combine_vec_kernel, n_rows, threads, 0, stream, a, na, (size_t)sa, b, nb, (size_t)sb, wa, wb, ca, cb, eps, out, dim);
+    LLM_CHECK_LAUNCH("pair_combine");
+    return LLM_OK;
+  }
   launch_kernel(pair_combine_kernel, n_rows, 256, 0, stream, a, na, (size_t)sa, b, nb, (size_t)sb, wa, wb, ca, cb, eps, out, dim);
   LLM_CHECK_LAUNCH("pair_combine");
   return LLM_OK;

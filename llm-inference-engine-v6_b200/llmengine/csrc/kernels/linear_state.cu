@@ -56,7 +56,7 @@ struct LinearStateParams {
   float* out;                                      // [tokens, H * dv]
   int H, G, dk, dv, R, tile;
   float q_scale, unit_eps;
-  int silu;      // q, k and v are silu of the sums
+  int silu;      // MODE 0: q, k and v are silu of the sums
   int walkers;   // threads of a block that hold the state (a multiple of 32 and of R); LS_FETCHERS more fetch
   int one_part;  // every product comes in one part
   int vec4;      // every row and column offset is a multiple of four numbers on a 16-byte boundary
@@ -267,8 +267,8 @@ __device__ __forceinline__ void fetch_issue(const LinearStateParams& p, size_t r
     for (int x = 0; x < U; ++x) {
       const int e = e0 + x * n_thr;
       if (e < n_qk) {
-        rows.q[e] = (p.silu ? silu_f(qv[x]) : qv[x]) * qmul;
-        rows.k[e] = p.silu ? silu_f(kv[x]) : kv[x];
+        rows.q[e] = (MODE == 0 && p.silu ? silu_f(qv[x]) : qv[x]) * qmul;
+        rows.k[e] = MODE == 0 && p.silu ? silu_f(kv[x]) : kv[x];
         if (MODE != 2) rows.a[e] = av[x];
       }
     }
@@ -288,7 +288,7 @@ __device__ __forceinline__ void fetch_issue(const LinearStateParams& p, size_t r
     }
 #pragma unroll
     for (int x = 0; x < U; ++x)
-      if (e0 + x * n_thr < n_v) rows.v[e0 + x * n_thr] = p.silu ? silu_f(vv[x]) : vv[x];
+      if (e0 + x * n_thr < n_v) rows.v[e0 + x * n_thr] = MODE == 0 && p.silu ? silu_f(vv[x]) : vv[x];
   }
   if (MODE == 2)
     for (int e = tid; e < 2 * cnt; e += n_thr) rows.a[e] = p.decay[(row0 + (e >> 1)) * p.decay_width + p.decay_off + (e & 1) * p.H + head];
@@ -301,7 +301,7 @@ __device__ __forceinline__ void fetch_finish(const LinearStateParams& p, int cnt
   const bool unit = MODE >= 2 && p.unit_eps >= 0.f;
   const float qmul = unit ? 1.0f : p.q_scale;
   const int n_qk = cnt * dkp;
-  if (p.one_part && p.silu) {  // the thread's own copies, as fetch_issue dealt them (a group of four numbers or one)
+  if (MODE == 0 && p.one_part && p.silu) {  // the thread's own copies, as fetch_issue dealt them (a group of four numbers or one)
     const int n_v = cnt * dv, V = p.vec4 ? 4 : 1;
     for (int e = tid * V; e < n_qk; e += n_thr * V)
       for (int i = e; i < e + V; ++i) {
@@ -684,8 +684,40 @@ __global__ void __launch_bounds__(128)
   }
 }
 
+template <int V>
+__device__ __forceinline__ void load_n(float (&x)[V], const float* p) {
+  if constexpr (V == 4) {
+    const float4 t = *reinterpret_cast<const float4*>(p);
+    x[0] = t.x; x[1] = t.y; x[2] = t.z; x[3] = t.w;
+  } else {
+#pragma unroll
+    for (int e = 0; e < V; ++e) x[e] = p[e];
+  }
+}
+template <int V>
+__device__ __forceinline__ void store_n(float* p, const float (&x)[V]) {
+  if constexpr (V == 4) *reinterpret_cast<float4*>(p) = make_float4(x[0], x[1], x[2], x[3]);
+  else
+#pragma unroll
+    for (int e = 0; e < V; ++e) p[e] = x[e];
+}
+template <int V>
+__device__ __forceinline__ void store_n(bf16* p, const float (&x)[V]) {
+  if constexpr (V == 4) {
+    const __nv_bfloat162 a = __floats2bfloat162_rn(x[0], x[1]), b = __floats2bfloat162_rn(x[2], x[3]);
+    uint2 u;
+    u.x = *reinterpret_cast<const uint32_t*>(&a);
+    u.y = *reinterpret_cast<const uint32_t*>(&b);
+    *reinterpret_cast<uint2*>(p) = u;
+  } else {
+#pragma unroll
+    for (int e = 0; e < V; ++e) p[e] = __float2bfloat16_rn(x[e]);
+  }
+}
+
 // The same for wide rows (all heads normed together): a block a (token, head), its numbers in the threads' turns, then block_sum.
-template <typename T>
+// V 4: rows of a multiple of four numbers on 16-byte boundaries, moved four at a time.
+template <typename T, int V>
 __global__ void __launch_bounds__(1024)
     wide_norm_gate_kernel(const float* __restrict__ o, const float* __restrict__ weight, int weight_per_head, const Sums gate, float eps,
                           T* __restrict__ out, int H, int dv, int sigmoid) {
@@ -696,15 +728,33 @@ __global__ void __launch_bounds__(1024)
   const int head = (int)(item - tok * H);
   const float* row = o + item * dv;
   float ss = 0.f;
-  for (int d = threadIdx.x; d < dv; d += blockDim.x) ss = fmaf(row[d], row[d], ss);
+  for (int d = threadIdx.x * V; d < dv; d += blockDim.x * V) {
+    float x[V];
+    load_n<V>(x, row + d);
+#pragma unroll
+    for (int e = 0; e < V; ++e) ss = fmaf(x[e], x[e], ss);
+  }
   const float inv = 1.0f / sqrtf(block_sum(ss, red) / (float)dv + eps);
-  for (int d = threadIdx.x; d < dv; d += blockDim.x) {
-    float v = row[d] * inv * weight[weight_per_head ? (size_t)head * dv + d : d];
-    if (gate.p) {
-      const float g = parts_sum(gate.p, gate.n, gate.stride, tok * gate.width + gate.off + (size_t)head * dv + d);
-      v *= (sigmoid ? 1.0f : g) / (1.0f + expf(-g));
+  for (int d = threadIdx.x * V; d < dv; d += blockDim.x * V) {
+    float x[V], w[V], g[V], t[V];
+    load_n<V>(x, row + d);
+    load_n<V>(w, weight + (weight_per_head ? (size_t)head * dv + d : d));
+    if (gate.p) {  // the parts in index order
+      const float* gp = gate.p + tok * gate.width + gate.off + (size_t)head * dv + d;
+      load_n<V>(g, gp);
+#pragma unroll 4
+      for (int k = 1; k < gate.n; ++k) {
+        load_n<V>(t, gp + (size_t)k * gate.stride);
+#pragma unroll
+        for (int e = 0; e < V; ++e) g[e] += t[e];
+      }
     }
-    out[item * dv + d] = from_f32<T>(v);
+#pragma unroll
+    for (int e = 0; e < V; ++e) {
+      x[e] = x[e] * inv * w[e];
+      if (gate.p) x[e] *= (sigmoid ? 1.0f : g[e]) / (1.0f + expf(-g[e]));
+    }
+    store_n<V>(out + item * dv + d, x);
   }
 }
 
@@ -786,6 +836,7 @@ extern "C" int llm_linear_state(int mode, const float* q, int qn, long long qs, 
   // the sums (before the query's scale)
   if (n_seqs == 0) return LLM_OK;
   LLM_REQUIRE(mode >= 0 && mode <= 3, "linear_state: unknown update rule %d", mode);
+  LLM_REQUIRE(!silu || mode == 0, "linear_state: activated sums go with the first rule");
   LLM_REQUIRE(n_seqs > 0 && n_seqs <= 65535 && H > 0 && H <= 65535 && G > 0 && H % G == 0 && dv > 0, "linear_state: bad sizes");
   LLM_REQUIRE(llm_linear_state_lanes(dk) > 0, "linear_state: a key size of %d is not in 1..%d", dk, 32 * KPT);
   LLM_REQUIRE(mode >= 2 || G == H, "linear_state: only the delta rules share query/key heads");
@@ -921,10 +972,15 @@ extern "C" int llm_head_norm_gate(const float* o, const float* weight, int weigh
     const int threads = min(1024, ceil_div(dv, 128) * 32);
     const long long rows = (long long)n_tokens * H;
     LLM_REQUIRE(rows <= 0x7fffffffLL, "head_norm_gate: too many rows");
-    if (dtype == LLM_F32)
-      launch_kernel(wide_norm_gate_kernel<float>, (int)rows, threads, 0, stream, o, weight, weight_per_head, g, eps, (float*)out, H, dv, sigmoid);
-    else
-      launch_kernel(wide_norm_gate_kernel<bf16>, (int)rows, threads, 0, stream, o, weight, weight_per_head, g, eps, (bf16*)out, H, dv, sigmoid);
+    auto quads = [](const void* q) { return ((uintptr_t)q & 15u) == 0; };
+    const bool vec = dv % 4 == 0 && gw % 4 == 0 && go % 4 == 0 && gs % 4 == 0 && quads(o) && quads(weight) && quads(gate) && quads(out);
+#define LLM_WIDE_NORM(T, V) \
+  launch_kernel(wide_norm_gate_kernel<T, V>, (int)rows, threads, 0, stream, o, weight, weight_per_head, g, eps, (T*)out, H, dv, sigmoid)
+    if (dtype == LLM_F32 && vec) LLM_WIDE_NORM(float, 4);
+    else if (dtype == LLM_F32) LLM_WIDE_NORM(float, 1);
+    else if (vec) LLM_WIDE_NORM(bf16, 4);
+    else LLM_WIDE_NORM(bf16, 1);
+#undef LLM_WIDE_NORM
     LLM_CHECK_LAUNCH("head_norm_gate");
     return LLM_OK;
   }

@@ -1425,7 +1425,7 @@ class CudaOps:
         ([parts, n, width] or [n, width]) read at column offsets, q and k with kv_heads heads of dk (head h reads head
         h // (heads / kv_heads)), v with heads of dv. decay: float32 rows; at decay_off a number per (head, key channel), or for
         "delta" [g: heads | beta: heads]; with decay_const a single row that holds for every token (decays that are constants
-        of the model); with silu, q, k and v are silu of their sums (q before its scale). out float32 [n, heads * dv]."""
+        of the model); with silu ("decay_write_read" alone), q, k and v are silu of their sums (q before its scale). out float32 [n, heads * dv]."""
         _need(decay, "linear_state.decay", torch.float32); _need(state, "linear_state.state", torch.float32); _need(out, "linear_state.out", torch.float32)
         assert decay.is_contiguous() and decay.dim() == 2 and state.is_contiguous() and out.is_contiguous() and out.shape[1] == heads * dv
         assert tuple(state.shape[1:]) == tuple(self.linear_state_shape(heads, dk, dv))

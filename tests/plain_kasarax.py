@@ -55,6 +55,9 @@ ROUNDING = None  # a function, or None. A 16-bit engine rounds the operands of i
 # of the weights: the difference to a run without it is the error that rounding alone causes.
 
 
+GAPS = None  # a list, or None: every routed layer adds, a token, the distance between its last chosen and first unchosen router logit
+
+
 def _r(x):
     return x if ROUNDING is None else ROUNDING(x)
 
@@ -207,6 +210,9 @@ def experts_ff(h, w, p, f):
     """Each token through the experts with the largest sigmoid scores; a score multiplies what its expert reads."""
     top = f["router"]["top"]
     scores = sigmoid(h @ w[p + "router"].t())
+    if GAPS is not None and top < f["router"]["experts"]:
+        z = torch.sort(h @ w[p + "router"].t(), dim=1, descending=True).values
+        GAPS.append(z[:, top - 1] - z[:, top])
     out = []
     for t in range(h.shape[0]):
         y = torch.zeros_like(h[t])
