@@ -625,7 +625,7 @@ def test_long_decoding_and_generation(model):
 @pytest.mark.parametrize("dt", DTYPES)
 @pytest.mark.parametrize("dim,vdim,conv", [(64, 32, 4), (32, 128, 3), (128, 64, 2), (48, 40, 3)])
 def test_single_tokens_behind_long_contexts(dt, dim, vdim, conv, tmp_path):
-    """Three requests of unequal length (up to 1,500 tokens) whose last tokens come one a step, side by side: single tokens whose
+    """Three requests of unequal length (up to 1,000 tokens) whose last tokens come one a step, side by side: single tokens whose
     key range is cut into pieces that run side by side and are merged, keys and values of different sizes, a learned sink and the added
     one where the pieces are merged, a gate a head behind them; a state and convolution inputs carried through it all."""
     layers = [layer("attention", att(4, 2, dim, vdim, 1.0 / dim ** 0.5, (0.3, 100)), dense(64)),
@@ -634,10 +634,10 @@ def test_single_tokens_behind_long_contexts(dt, dim, vdim, conv, tmp_path):
     cfg = config(120, 64, 1e-5, 0.7, layers, 2048)
     d = write_model(str(tmp_path / "m"), cfg, dt, sharp=True)
     pc, pw = P.read_model(d)
-    reqs = {"a": random_ids(1500, 120, 1), "b": random_ids(700, 120, 2), "c": random_ids(200, 120, 3)}
-    tail = 24
+    reqs = {"a": random_ids(1000, 120, 1), "b": random_ids(500, 120, 2), "c": random_ids(120, 120, 3)}
+    tail = 12
     eng = llmengine.Engine(d, NAMES[dt], block_size=16)
-    eng.configure_cache(num_blocks=(1536 + 704 + 256) // 16, block_size=16, num_slots=4)
+    eng.configure_cache(num_blocks=(1024 + 512 + 128) // 16, block_size=16, num_slots=4)
     ids = {"a": 1, "b": 2, "c": 3}
     for k, v in reqs.items():
         eng.run_step([(ids[k], v[:-tail], [])], end=[])
